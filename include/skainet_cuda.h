@@ -51,6 +51,7 @@ extern "C" {
 #define SKAINET_ENC_Q4_K  12   /* ggml Q4_K: 144-byte super-blocks of 256                             */
 #define SKAINET_ENC_Q5_K  13   /* ggml Q5_K: 176-byte super-blocks of 256                             */
 #define SKAINET_ENC_Q6_K  14   /* ggml Q6_K: 210-byte super-blocks of 256                             */
+#define SKAINET_ENC_BF16  30   /* bfloat16 elements, row-major only (ggml type id 30)                   */
 
 /* Byte order of a packed [out, in] weight handed to upload (KernelKey layout classes,
  * skainet-backends/skainet-backend-api/src/commonMain/kotlin/sk/ainet/backend/api/kernel/KernelKey.kt:77-90). */

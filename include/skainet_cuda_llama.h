@@ -26,6 +26,9 @@
 extern "C" {
 #endif
 
+/* A model of any design this runtime holds. llama_create makes the Llama-style one, skainet_cuda_tivazen.h declares another;
+ * free, finalize, reset, reset_seq, prefill, forward, fake_prefill, decode, generate, logits, step_cost, peek and stream take
+ * either, create / set_weight / set_norm / synth / get_weight / tp_* are the Llama-style model's own. */
 typedef int64_t skainet_model_t;
 
 typedef struct {
@@ -76,12 +79,18 @@ SKAINET_CUDA_API int32_t skainet_cuda_llama_finalize(skainet_model_t m);
 SKAINET_CUDA_API int32_t skainet_cuda_llama_tp_unique_id(uint8_t* id128);
 SKAINET_CUDA_API int32_t skainet_cuda_llama_tp_init(skainet_model_t m, const uint8_t* id128);
 
-/* Forget all cached tokens of every sequence. */
+/* Forget all cached tokens of every sequence / of one sequence, whose slot is then free for another. */
 SKAINET_CUDA_API int32_t skainet_cuda_llama_reset(skainet_model_t m);
+SKAINET_CUDA_API int32_t skainet_cuda_llama_reset_seq(skainet_model_t m, int32_t seq);
 /* Runs n prompt tokens of sequence `seq` through the model, filling its cache from its current
  * position. If next_token_host != NULL it receives the greedy token after the last prompt token. */
 SKAINET_CUDA_API int32_t skainet_cuda_llama_prefill(skainet_model_t m, int32_t seq, const int32_t* tokens_host, int32_t n,
     int32_t* next_token_host);
+/* Runs the next n given tokens of sequence `seq` (a prompt portion, or one decoded token through the captured step) and
+ * returns the logits after the n_want places listed in want_host (indices into the n tokens, any order, repeats allowed):
+ * logits_host[n_want][vocab]. Sequences longer than one prompt pass are cut inside. Single-GPU models. */
+SKAINET_CUDA_API int32_t skainet_cuda_llama_forward(skainet_model_t m, int32_t seq, const int32_t* tokens_host, int32_t n,
+    const int32_t* want_host, int32_t n_want, float* logits_host);
 /* Fills sequence `seq`'s cache with n tokens worth of seeded random K/V instead of running a prompt
  * (throughput runs at long context, where the reference CPU path could not produce the prefill). */
 SKAINET_CUDA_API int32_t skainet_cuda_llama_fake_prefill(skainet_model_t m, int32_t seq, int32_t n, uint64_t seed);

@@ -13,10 +13,10 @@ LIB_PATH = os.path.join(HERE, "libskainet_cuda.so")
 
 OK = 0
 ERR_INVALID, ERR_CUDA, ERR_NODEVICE, ERR_OOM, ERR_HANDLE, ERR_TIMEOUT, ERR_COMM = -1, -2, -3, -4, -5, -6, -7
-ENC = {"Q8_0": 8, "Q4_K": 12, "Q5_K": 13, "Q6_K": 14}
+ENC = {"Q8_0": 8, "Q4_K": 12, "Q5_K": 13, "Q6_K": 14, "BF16": 30}
 ENC_NAME = {v: k for k, v in ENC.items()}
-BLOCK_BYTES = {"Q8_0": 34, "Q4_K": 144, "Q5_K": 176, "Q6_K": 210}
-BLOCK_ELEMS = {"Q8_0": 32, "Q4_K": 256, "Q5_K": 256, "Q6_K": 256}
+BLOCK_BYTES = {"Q8_0": 34, "Q4_K": 144, "Q5_K": 176, "Q6_K": 210, "BF16": 2}
+BLOCK_ELEMS = {"Q8_0": 32, "Q4_K": 256, "Q5_K": 256, "Q6_K": 256, "BF16": 1}
 ORDER_ROW_MAJOR, ORDER_INPUT_MAJOR = 0, 1
 ACT_NATIVE, ACT_F32 = 0, 1
 
@@ -107,7 +107,9 @@ SIGNATURES = {
     "skainet_cuda_llama_tp_unique_id": [C.POINTER(C.c_uint8)],
     "skainet_cuda_llama_tp_init": [i64, C.POINTER(C.c_uint8)],
     "skainet_cuda_llama_reset": [i64],
+    "skainet_cuda_llama_reset_seq": [i64, i32],
     "skainet_cuda_llama_prefill": [i64, i32, i32p, i32, i32p],
+    "skainet_cuda_llama_forward": [i64, i32, i32p, i32, i32p, i32, f32p],
     "skainet_cuda_llama_fake_prefill": [i64, i32, i32, C.c_uint64],
     "skainet_cuda_llama_decode": [i64, i32, i32p, i32p],
     "skainet_cuda_llama_generate": [i64, i32, i32p, i32, i32p],
@@ -116,6 +118,11 @@ SIGNATURES = {
     "skainet_cuda_llama_peek": [i64, i32, f32p, i64],
     "skainet_cuda_llama_tp_exchange_time": [i64, i32, i32, i32, f32p],
     "skainet_cuda_llama_stream": [i64, C.POINTER(vp)],
+    # include/skainet_cuda_tivazen.h
+    "skainet_cuda_tivazen_create": [vp, vp, i64p],
+    "skainet_cuda_tivazen_set_weight": [i64, i32, i32, i32, i64],
+    "skainet_cuda_tivazen_set_vector": [i64, i32, i32, f32p, i32],
+    "skainet_cuda_tivazen_synth": [i64, C.c_uint64, f32],
 }
 _RESTYPE = {"skainet_cuda_last_error": C.c_char_p, "skainet_cuda_version": C.c_char_p}
 

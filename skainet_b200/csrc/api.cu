@@ -2,6 +2,7 @@
 // the resident-weight registry, per-stream scratch, and the host-pointer twins of the reference's
 // native entry points, which are thin wrappers over the resident API (upload, run, read back).
 #include "common.cuh"
+#include "linear_bf16.cuh"
 #include <cstdlib>
 #include "matvec_fused.cuh"
 
@@ -166,11 +167,13 @@ int32_t weight_alloc(int enc, int rows, int cols, Weight** out) {
         case SKAINET_ENC_Q8_0: s_qs = nb * 32; s_hdr = nb * 2; break;
         case SKAINET_ENC_Q4_K: s_qs = nb * 128; s_hdr = nb * 16; break;
         case SKAINET_ENC_Q5_K: s_qs = nb * 128; s_hdr = nb * 16; s_extra = nb * 32; break;
+        case SKAINET_ENC_BF16: s_qs = (size_t) rows * bf16_ld(cols) * 2; break;
         default:               s_qs = nb * 128; s_hdr = nb * 16; s_extra = nb * 64; s_aux = nb * 2; break;
     }
     const size_t total = a256(s_qs) + a256(s_hdr) + a256(s_extra) + a256(s_aux) + 256;
     cudaError_t e = cudaMalloc(&w->base, total);
     if (e != cudaSuccess) { delete w; return cuda_fail(e, "cudaMalloc(weight)", __FILE__, __LINE__); }
+    if (enc == SKAINET_ENC_BF16) cudaMemset(w->base, 0, total);      // the row tails stay zero
     uint8_t* p = (uint8_t*) w->base;
     w->qs = p; p += a256(s_qs);
     w->hdr = p; p += a256(s_hdr);
@@ -356,6 +359,7 @@ static int32_t weight_build(const uint8_t* bytes, bool on_device, int64_t nbytes
     *out = 0;
     SK_TRY(validate_geometry(enc, rows, cols, "weight_upload"));
     SK_REQUIRE(order == SKAINET_ORDER_ROW_MAJOR || order == SKAINET_ORDER_INPUT_MAJOR, "weight_upload: unknown order %d", order);
+    SK_REQUIRE(enc != SKAINET_ENC_BF16 || order == SKAINET_ORDER_ROW_MAJOR, "weight_upload: BF16 weights are row-major");
     const int64_t need = (int64_t) rows * (cols / block_elems(enc)) * block_bytes(enc);
     SK_REQUIRE(nbytes == need, "weight_upload: %lld bytes given, [%d, %d] needs %lld", (long long) nbytes, rows, cols, (long long) need);
     SK_REQUIRE(need == 0 || bytes != nullptr, "weight_upload: null bytes");
@@ -402,7 +406,7 @@ int32_t skainet_cuda_weight_synth(int32_t enc, int32_t rows, int32_t cols, uint6
     SK_REQUIRE(out != nullptr, "weight_synth: null output");
     *out = 0;
     SK_TRY(validate_geometry(enc, rows, cols, "weight_synth"));
-    SK_REQUIRE(enc == SKAINET_ENC_Q4_K || enc == SKAINET_ENC_Q8_0, "weight_synth: encoding %d not supported", enc);
+    SK_REQUIRE(enc == SKAINET_ENC_Q4_K || enc == SKAINET_ENC_Q8_0 || (enc == SKAINET_ENC_BF16 && mode == 0), "weight_synth: encoding %d not supported in mode %d", enc, mode);
     SK_REQUIRE(mode == 0 || mode == 1, "weight_synth: mode %d", mode);
     Weight* w = nullptr;
     SK_TRY(weight_alloc(enc, rows, cols, &w));
@@ -471,6 +475,16 @@ int32_t skainet_cuda_matmul_dev(skainet_weight_t h, const float* x_dev, int32_t 
     SK_TRY(ensure_device());
     cudaStream_t s = as_stream(stream);
     if (w->cols == 0) { SK_CUDA(cudaMemsetAsync(y_dev, 0, sizeof(float) * (size_t) m * w->rows, s)); return SKAINET_CUDA_OK; }
+    if (w->enc == SKAINET_ENC_BF16) {          // bf16 activations with fp32 accumulation, or fp32 throughout in the F32 mode
+        LinearArgs l;
+        l.f32_act = act_mode == SKAINET_ACT_F32;
+        l.ldw = l.ldx = bf16_ld(w->cols);
+        void* act = nullptr;
+        SK_TRY(scratch_get(s, SCRATCH_ACT, (size_t) m * l.ldx * (l.f32_act ? 4 : 2), &act));
+        SK_TRY(launch_to_act(x_dev, m, w->cols, act, l.ldx, l.f32_act, s));
+        l.w = (const bf16*) w->qs; l.w_rows = w->rows; l.x = act; l.x_rows_alloc = l.rows = m; l.y = y_dev; l.ldy = w->rows;
+        return launch_linear_bf16(l, s);
+    }
     // One activation row of a Q4_K weight of 4 MB or more: a single launch, the ring kernel quantizes the row in its own
     // prologue (once per SM) while the first weight stages are in flight (config 2: 5.7 / 7.2 us per matvec against
     // 8.0 / 8.4 us for a quantizer launch followed by the matvec).
@@ -498,6 +512,7 @@ int32_t skainet_cuda_matmul_dev(skainet_weight_t h, const float* x_dev, int32_t 
 int32_t skainet_cuda_probe_read_dev(skainet_weight_t h, skainet_stream_t stream) {
     Weight* w = weight_from_handle(h);
     if (!w) return SKAINET_CUDA_ERR_HANDLE;
+    SK_REQUIRE(w->enc != SKAINET_ENC_BF16, "probe_read: packed encodings only");
     SK_TRY(ensure_device());
     void* sink = nullptr;
     SK_TRY(scratch_get(as_stream(stream), SCRATCH_FUSED2, 64, &sink));
@@ -512,6 +527,7 @@ int32_t skainet_cuda_matvec_fused_dev(skainet_weight_t h, const float* x_dev, co
     SK_REQUIRE(x_dev != nullptr && y_dev != nullptr, "matvec_fused: null activation or output");
     SK_REQUIRE((((uintptr_t) x_dev | (uintptr_t) gamma_dev) & 15) == 0, "matvec_fused: x and gamma must be 16-byte aligned");
     SK_REQUIRE(w->cols > 0, "matvec_fused: empty input dimension");
+    SK_REQUIRE(w->enc != SKAINET_ENC_BF16, "matvec_fused: encoding %d not supported", w->enc);
     SK_TRY(ensure_device());
     cudaStream_t s = as_stream(stream);
     MatvecIn in; in.x = x_dev; in.gamma = gamma_dev; in.eps = eps;

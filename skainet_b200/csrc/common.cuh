@@ -40,13 +40,14 @@ int32_t ensure_device();   // SKAINET_CUDA_OK once a usable sm_100 device is cur
 inline cudaStream_t as_stream(skainet_stream_t s) { return reinterpret_cast<cudaStream_t>(s); }
 
 // ---- block geometry ----------------------------------------------------------------------------
-inline int block_elems(int enc) { return enc == SKAINET_ENC_Q8_0 ? 32 : 256; }
+inline int block_elems(int enc) { return enc == SKAINET_ENC_Q8_0 ? 32 : enc == SKAINET_ENC_BF16 ? 1 : 256; }
 inline int block_bytes(int enc) {
     switch (enc) {
         case SKAINET_ENC_Q8_0: return 34;
         case SKAINET_ENC_Q4_K: return 144;
         case SKAINET_ENC_Q5_K: return 176;
         case SKAINET_ENC_Q6_K: return 210;
+        case SKAINET_ENC_BF16: return 2;
         default: return 0;
     }
 }
@@ -58,6 +59,7 @@ inline int block_bytes(int enc) {
 //   Q4_K: qs     u8   [rows][cols/256][128]        hdr 16 B   [rows][cols/256]  (d, dmin, 12 scale bytes)
 //   Q5_K: qs as Q4_K, hdr as Q4_K,                 extra qh   [rows][cols/256][32]
 //   Q6_K: ql     u8   [rows][cols/256][128]        hdr 16 B = 16 int8 scales; extra: qh [..][64] ; d f16 plane in aux
+//   BF16: elements, [rows][ld] with ld = cols rounded up to 64 and a zero tail (bf16_ld, linear_bf16.cuh)
 // The split is a pure byte permutation: export() restores the canonical bytes exactly.
 struct Weight {
     int32_t enc = 0, rows = 0, cols = 0, bpr = 0;  // bpr = blocks per row

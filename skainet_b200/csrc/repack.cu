@@ -6,6 +6,7 @@
 // product and difference individually rounded (__fmul_rn/__fsub_rn: no FMA contraction), which is
 // what makes the output bit-identical to the JVM's strict binary32 arithmetic.
 #include "common.cuh"
+#include "linear_bf16.cuh"
 
 namespace sk {
 
@@ -51,7 +52,15 @@ __global__ void plane_permute_kernel(uint16_t* canon, uint16_t* qs, uint16_t* hd
     }
 }
 
+// BF16 rows are only re-pitched.
+static int32_t copy_bf16_rows(void* dst, size_t dst_ld, const void* src, size_t src_ld, int rows, int cols, cudaStream_t s) {
+    if (rows == 0 || cols == 0) return SKAINET_CUDA_OK;
+    SK_CUDA(cudaMemcpy2DAsync(dst, dst_ld * 2, src, src_ld * 2, (size_t) cols * 2, rows, cudaMemcpyDeviceToDevice, s));
+    return SKAINET_CUDA_OK;
+}
+
 int32_t launch_split_planes(const uint8_t* canon_dev, Weight& w, int order, cudaStream_t s) {
+    if (w.enc == SKAINET_ENC_BF16) return copy_bf16_rows(w.qs, bf16_ld(w.cols), canon_dev, w.cols, w.rows, w.cols, s);
     const int bb2 = block_bytes(w.enc) / 2;
     const int64_t total = (int64_t) w.rows * w.bpr * bb2;
     if (total == 0) return SKAINET_CUDA_OK;
@@ -63,6 +72,7 @@ int32_t launch_split_planes(const uint8_t* canon_dev, Weight& w, int order, cuda
 }
 
 int32_t launch_join_planes(const Weight& w, uint8_t* canon_dev, cudaStream_t s) {
+    if (w.enc == SKAINET_ENC_BF16) return copy_bf16_rows(canon_dev, w.cols, w.qs, bf16_ld(w.cols), w.rows, w.cols, s);
     const int bb2 = block_bytes(w.enc) / 2;
     const int64_t total = (int64_t) w.rows * w.bpr * bb2;
     if (total == 0) return SKAINET_CUDA_OK;
@@ -116,8 +126,11 @@ __device__ float decode_elem(int enc, const uint8_t* qs, const uint8_t* hdr, con
     }
 }
 
+__device__ __forceinline__ float bf16_bits_to_float(uint16_t h) { return __uint_as_float((uint32_t) h << 16); }
+
 __device__ __forceinline__ float decode_at(const WView& w, int64_t pblk, int e) {
     switch (w.enc) {
+        case SKAINET_ENC_BF16: return bf16_bits_to_float(((const uint16_t*) w.qs)[pblk / w.cols * bf16_ld(w.cols) + pblk % w.cols]);
         case SKAINET_ENC_Q8_0: return decode_elem(w.enc, w.qs + pblk * 32, w.hdr + pblk * 2, nullptr, nullptr, e);
         case SKAINET_ENC_Q4_K: return decode_elem(w.enc, w.qs + pblk * 128, w.hdr + pblk * 16, nullptr, nullptr, e);
         case SKAINET_ENC_Q5_K: return decode_elem(w.enc, w.qs + pblk * 128, w.hdr + pblk * 16, w.extra + pblk * 32, nullptr, e);
@@ -126,7 +139,7 @@ __device__ __forceinline__ float decode_at(const WView& w, int64_t pblk, int e) 
 }
 
 __global__ void dequant_weight_kernel(WView w, float* out) {
-    const int be = w.enc == SKAINET_ENC_Q8_0 ? 32 : 256;
+    const int be = w.enc == SKAINET_ENC_Q8_0 ? 32 : w.enc == SKAINET_ENC_BF16 ? 1 : 256;
     const int64_t total = (int64_t) w.rows * w.cols;
     for (int64_t i = blockIdx.x * (int64_t) blockDim.x + threadIdx.x; i < total; i += (int64_t) gridDim.x * blockDim.x)
         out[i] = decode_at(w, i / be, (int) (i % be));
@@ -143,7 +156,7 @@ int32_t launch_dequant_weight(const Weight& w, float* out, cudaStream_t s) {
 
 // Canonical (un-split) blocks straight to floats: the twin of DequantOps.dequant*FromBytes.
 __global__ void dequant_canonical_kernel(int enc, const uint8_t* canon, int64_t nblocks, float* out) {
-    const int be = enc == SKAINET_ENC_Q8_0 ? 32 : 256;
+    const int be = enc == SKAINET_ENC_Q8_0 ? 32 : enc == SKAINET_ENC_BF16 ? 1 : 256;
     const int64_t total = nblocks * be;
     for (int64_t i = blockIdx.x * (int64_t) blockDim.x + threadIdx.x; i < total; i += (int64_t) gridDim.x * blockDim.x) {
         const int64_t blk = i / be; const int e = (int) (i % be);
@@ -152,6 +165,7 @@ __global__ void dequant_canonical_kernel(int enc, const uint8_t* canon, int64_t 
         switch (enc) {
             case SKAINET_ENC_Q8_0: p = canon + blk * 34;  v = decode_elem(enc, p + 2, p, nullptr, nullptr, e); break;
             case SKAINET_ENC_Q4_K: p = canon + blk * 144; v = decode_elem(enc, p + 16, p, nullptr, nullptr, e); break;
+            case SKAINET_ENC_BF16: v = bf16_bits_to_float(((const uint16_t*) canon)[blk]); break;
             case SKAINET_ENC_Q5_K: p = canon + blk * 176; v = decode_elem(enc, p + 48, p, p + 16, nullptr, e); break;
             default:               p = canon + blk * 210; v = decode_elem(enc, p, p + 192, p + 128, p + 208, e); break;
         }
@@ -172,7 +186,7 @@ int32_t launch_dequant_canonical(int enc, const uint8_t* canon_dev, int64_t nblo
 __global__ void embed_kernel(WView w, const int32_t* ids, int n, float* out) {
     const int i = blockIdx.x;
     const int row = ids[i];
-    const int be = w.enc == SKAINET_ENC_Q8_0 ? 32 : 256;
+    const int be = w.enc == SKAINET_ENC_Q8_0 ? 32 : w.enc == SKAINET_ENC_BF16 ? 1 : 256;
     for (int c = threadIdx.x; c < w.cols; c += blockDim.x) {
         float v = 0.0f;
         if (row >= 0 && row < w.rows) v = decode_at(w, (int64_t) row * w.bpr + c / be, c % be);
@@ -310,6 +324,14 @@ __global__ void synth_q8_0_kernel(int8_t* codes, __half* scales, int64_t nblocks
     }
 }
 
+__global__ void synth_bf16_kernel(bf16* w, int rows, int cols, int ld, uint64_t seed, float std, int64_t row0, int64_t col0, int64_t full_cols) {
+    const int64_t total = (int64_t) rows * cols;
+    for (int64_t i = blockIdx.x * (int64_t) blockDim.x + threadIdx.x; i < total; i += (int64_t) gridDim.x * blockDim.x) {
+        const int64_t r = i / cols, c = i % cols;
+        w[r * ld + c] = __float2bfloat16_rn(std * normal_at(seed, (uint64_t) ((row0 + r) * full_cols + col0 + c)));
+    }
+}
+
 int32_t launch_synth(Weight& w, uint64_t seed, float std, int mode, int64_t row0, int64_t col0, int64_t full_cols, cudaStream_t s) {
     const int64_t nblocks = (int64_t) w.rows * w.bpr;
     if (nblocks == 0) return SKAINET_CUDA_OK;
@@ -317,6 +339,7 @@ int32_t launch_synth(Weight& w, uint64_t seed, float std, int mode, int64_t row0
     if (full_cols <= 0) full_cols = w.cols;
     if (w.enc == SKAINET_ENC_Q4_K) synth_q4k_kernel<<<grid, 256, 0, s>>>(w.qs, w.hdr, nblocks, seed, std, mode, w.bpr, row0, col0, full_cols);
     else if (w.enc == SKAINET_ENC_Q8_0) synth_q8_0_kernel<<<grid, 256, 0, s>>>((int8_t*) w.qs, (__half*) w.hdr, nblocks, seed, std, mode, w.bpr, row0, col0, full_cols);
+    else if (w.enc == SKAINET_ENC_BF16) synth_bf16_kernel<<<148 * 16, 256, 0, s>>>((bf16*) w.qs, w.rows, w.cols, bf16_ld(w.cols), seed, std, row0, col0, full_cols);
     else { set_error("weight_synth: encoding %d not supported", w.enc); return SKAINET_CUDA_ERR_INVALID; }
     SK_CUDA(cudaGetLastError());
     return SKAINET_CUDA_OK;

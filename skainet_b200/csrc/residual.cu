@@ -1,0 +1,172 @@
+// Residual, one-number norm and depth average (contract: residual.cuh). All HBM- or latency-bound: one pass over the row for
+// the sum of squares, one that writes. With few rows a cluster of up to eight CTAs shares a row (the sum of squares through
+// distributed shared memory), because a late layer's average reads every earlier state of the row.
+#include "residual.cuh"
+#include "tma.cuh"
+
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
+namespace sk {
+
+namespace {
+
+constexpr int RT = 256;
+
+__device__ __forceinline__ float block_sum(float v, float* sh) {
+    v = skd::warp_sum(v);
+    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.0f;
+    for (int i = 0; i < RT / 32; ++i) t += sh[i];
+    __syncthreads();
+    return t;
+}
+
+// V = 4: cols and every stride are multiples of four; V = 1: any.
+template <int V> struct Vec { float v[V]; };
+template <int V> __device__ __forceinline__ Vec<V> ld(const float* p) {
+    Vec<V> r;
+    if (V == 4) { const float4 q = *reinterpret_cast<const float4*>(p); r.v[0] = q.x; r.v[V > 1 ? 1 : 0] = q.y; r.v[V > 2 ? 2 : 0] = q.z; r.v[V > 3 ? 3 : 0] = q.w; }
+    else r.v[0] = *p;
+    return r;
+}
+template <int V> __device__ __forceinline__ void st(float* p, const Vec<V>& r) {
+    if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[V > 1 ? 1 : 0], r.v[V > 2 ? 2 : 0], r.v[V > 3 ? 3 : 0]);
+    else *p = r.v[0];
+}
+template <int V> __device__ __forceinline__ void st_act(float* p, const Vec<V>& r) { st<V>(p, r); }
+template <int V> __device__ __forceinline__ void st_act(bf16* p, const Vec<V>& r) {
+    if (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(skd::pack_bf16(r.v[0], r.v[V > 1 ? 1 : 0]), skd::pack_bf16(r.v[V > 2 ? 2 : 0], r.v[V > 3 ? 3 : 0]));
+    else *p = __float2bfloat16_rn(r.v[0]);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(RT) sublayer_kernel(const SublayerArgs a) {
+    namespace cg = cooperative_groups;
+    extern __shared__ __align__(16) float sy[];                 // this CTA's part of the sublayer output
+    __shared__ float sh[RT / 32], part;
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    cg::cluster_group cl = cg::this_cluster();
+    const int cs = (int) cl.num_blocks(), rank = (int) cl.block_rank(), row = blockIdx.x / cs;
+    const int per = ((a.cols + cs - 1) / cs + 3) / 4 * 4, c0 = min(a.cols, rank * per), c1 = min(a.cols, c0 + per);
+    float ss = 0.0f;
+    for (int c = c0 + (int) threadIdx.x * V; c < c1; c += RT * V) {
+        Vec<V> v;
+        if (a.slot_pos) {
+            v = ld<V>(a.y + (size_t) a.slot_pos[(size_t) row * a.top] * a.cols + c);
+            for (int k = 1; k < a.top; ++k) {
+                const Vec<V> u = ld<V>(a.y + (size_t) a.slot_pos[(size_t) row * a.top + k] * a.cols + c);
+#pragma unroll
+                for (int i = 0; i < V; ++i) v.v[i] += u.v[i];
+            }
+        } else v = ld<V>(a.y + (size_t) row * a.cols + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss += v.v[i] * v.v[i];
+        st<V>(sy + c - c0, v);
+    }
+    ss = block_sum(ss, sh);
+    if (cs > 1) {
+        if (threadIdx.x == 0) part = ss;
+        cl.sync();
+        ss = 0.0f;
+        for (int i = 0; i < cs; ++i) ss += *cl.map_shared_rank(&part, i);
+    }
+    const float r = 1.0f / sqrtf(ss / (float) a.cols + a.eps) * a.gain;
+    const size_t at = (size_t) row * a.cols;
+    for (int c = c0 + (int) threadIdx.x * V; c < c1; c += RT * V) {
+        Vec<V> v = ld<V>(a.base + at + c);
+        const Vec<V> y = ld<V>(sy + c - c0);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v.v[i] += y.v[i] * r;
+        st<V>(a.state + at + c, v);
+        if (a.n_states > 0) {
+            Vec<V> x;
+            const float cl_ = a.coef[a.n_states - 1];
+#pragma unroll
+            for (int i = 0; i < V; ++i) x.v[i] = cl_ * v.v[i];
+#pragma unroll 8
+            for (int j = 0; j < a.n_states - 1; ++j) {
+                const Vec<V> s = ld<V>(a.states + (size_t) j * a.state_stride + at + c);
+                const float f = a.coef[j];
+#pragma unroll
+                for (int i = 0; i < V; ++i) x.v[i] = fmaf(f, s.v[i], x.v[i]);
+            }
+            st<V>(a.x + at + c, x);
+            v = x;
+        }
+        st_act<V>((T*) a.act + (size_t) row * a.act_ld + c, v);
+    }
+    if (cs > 1) cl.sync();                                      // no CTA leaves while its partial sum may still be read
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RT) embed_rows_kernel(const bf16* __restrict__ table, int ld_, const int32_t* __restrict__ ids, int cols, int vocab,
+                                                        float* __restrict__ x, float* __restrict__ state0, T* __restrict__ act, int act_ld) {
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    const int row = blockIdx.x, id = min(max(ids[row], 0), vocab - 1);
+    for (int c = threadIdx.x; c < cols; c += RT) {
+        const float v = __bfloat162float(table[(size_t) id * ld_ + c]);
+        x[(size_t) row * cols + c] = v; state0[(size_t) row * cols + c] = v;
+        skd::store_act(act + (size_t) row * act_ld + c, v);
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RT) scalar_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ index, int cols, float gain, float eps,
+                                                         T* __restrict__ act, int act_ld) {
+    __shared__ float sh[RT / 32];
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    const float* p = x + (size_t) (index ? index[blockIdx.x] : (int) blockIdx.x) * cols;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < cols; c += RT) ss += p[c] * p[c];
+    ss = block_sum(ss, sh);
+    const float r = 1.0f / sqrtf(ss / (float) cols + eps) * gain;
+    for (int c = threadIdx.x; c < cols; c += RT) skd::store_act(act + (size_t) blockIdx.x * act_ld + c, p[c] * r);
+}
+
+template <typename T, int V>
+int32_t run_sublayer(const SublayerArgs& a, cudaStream_t s) {
+    int cs = 1;                                                 // CTAs per row: while the machine has room and a CTA keeps 256 columns
+    while (cs < 8 && a.rows * cs * 2 <= sm_count() && a.cols / (cs * 2) >= 256) cs *= 2;
+    const int per = ((a.cols + cs - 1) / cs + 3) / 4 * 4;
+    SK_TRY(ensure_dynamic_smem((const void*) sublayer_kernel<T, V>, per * (int) sizeof(float)));
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.rows * cs); cfg.blockDim = dim3(RT); cfg.dynamicSmemBytes = per * sizeof(float); cfg.stream = s;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = 1;
+    at[1].id = cudaLaunchAttributeClusterDimension; at[1].val.clusterDim.x = cs; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
+    cfg.attrs = at; cfg.numAttrs = 2;
+    SK_CUDA(cudaLaunchKernelEx(&cfg, sublayer_kernel<T, V>, a));
+    return SKAINET_CUDA_OK;
+}
+
+}  // namespace
+
+int32_t launch_sublayer(const SublayerArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return SKAINET_CUDA_OK;
+    const bool vec = a.cols % 4 == 0 && a.act_ld % 4 == 0 && a.state_stride % 4 == 0;
+    if (a.f32_act) return vec ? run_sublayer<float, 4>(a, s) : run_sublayer<float, 1>(a, s);
+    return vec ? run_sublayer<bf16, 4>(a, s) : run_sublayer<bf16, 1>(a, s);
+}
+
+int32_t launch_embed_rows(const bf16* table, int ld_, const int32_t* ids, int rows, int cols, int vocab, float* x, float* state0, void* act, int act_ld,
+                          bool f32_act, cudaStream_t s) {
+    if (rows <= 0) return SKAINET_CUDA_OK;
+    if (f32_act) SK_CUDA(launch_pdl(embed_rows_kernel<float>, dim3(rows), dim3(RT), 0, s, table, ld_, ids, cols, vocab, x, state0, (float*) act, act_ld));
+    else SK_CUDA(launch_pdl(embed_rows_kernel<bf16>, dim3(rows), dim3(RT), 0, s, table, ld_, ids, cols, vocab, x, state0, (bf16*) act, act_ld));
+    return SKAINET_CUDA_OK;
+}
+
+int32_t launch_scalar_norm(const float* x, const int32_t* index, int rows, int cols, float gain, float eps, void* act, int act_ld, bool f32_act, cudaStream_t s) {
+    if (rows <= 0) return SKAINET_CUDA_OK;
+    if (f32_act) SK_CUDA(launch_pdl(scalar_norm_kernel<float>, dim3(rows), dim3(RT), 0, s, x, index, cols, gain, eps, (float*) act, act_ld));
+    else SK_CUDA(launch_pdl(scalar_norm_kernel<bf16>, dim3(rows), dim3(RT), 0, s, x, index, cols, gain, eps, (bf16*) act, act_ld));
+    return SKAINET_CUDA_OK;
+}
+
+}  // namespace sk

@@ -2,6 +2,7 @@
 // a graph executor's fused-op handlers call: fused_qkv_proj and fused_swiglu_ffn
 // (skainet-compile/skainet-compile-opt/src/commonMain/kotlin/sk/ainet/compile/opt/passes/LLMFusionPass.kt:17-23,86,117;
 // CPU decompositions in skainet-compile/skainet-compile-dag/src/commonMain/kotlin/sk/ainet/lang/graph/exec/LLMFusedOpHandlers.kt:27-68,86-196).
+#include "linear_bf16.cuh"
 #include "stepops.cuh"
 #include "tma.cuh"
 #include "matvec_fused.cuh"
@@ -139,6 +140,13 @@ int32_t weight_concat_rows(const Weight* a, const Weight* b, const Weight* c, We
     SK_TRY(weight_alloc(a->enc, rows, a->cols, out));
     Weight* w = *out;
     const Weight* parts[3] = {a, b, c};
+    if (a->enc == SKAINET_ENC_BF16) {
+        const size_t row_bytes = (size_t) bf16_ld(a->cols) * 2;
+        size_t at = 0;
+        for (const Weight* p : parts)
+            if (p) { SK_CUDA(cudaMemcpy(w->qs + at, p->qs, p->rows * row_bytes, cudaMemcpyDeviceToDevice)); at += p->rows * row_bytes; }
+        return SKAINET_CUDA_OK;
+    }
     // bytes per block of each plane (see the Weight record): main codes, header / scales, extra bit plane, aux scale plane
     size_t pb[4] = {128, 16, 0, 0};
     if (a->enc == SKAINET_ENC_Q8_0) { pb[0] = 32; pb[1] = 2; }

@@ -1,13 +1,13 @@
-"""Host-side handle of the decoder runtime inside libskainet_cuda (include/skainet_cuda_llama.h)."""
+"""Host-side handle of the Llama-style design of the decoder runtime inside libskainet_cuda (include/skainet_cuda_llama.h)."""
 from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import Optional, Sequence
 
 import numpy as np
 
 from . import _lib as L
+from .decoder import Decoder
 from .device import Weight
 
 W_EMBED, W_HEAD, W_OUT_NORM, W_ATTN_NORM, W_Q, W_K, W_V, W_O, W_FFN_NORM, W_GATE, W_UP, W_DOWN, W_QKV, W_GATE_UP = range(14)
@@ -55,13 +55,39 @@ class LlamaConfig:
                        L.ENC[self.table_enc], self.tp_rank, self.tp_world)
 
 
-class Llama:
+class Llama(Decoder):
     def __init__(self, cfg: LlamaConfig):
         self.cfg = cfg
         h = C.c_int64()
         c = cfg.to_c()
         L.check(L.lib().skainet_cuda_llama_create(C.byref(c), C.byref(h)))
-        self.handle = h.value
+        super().__init__(h.value, cfg.vocab, cfg.max_seq, cfg.max_batch)
+
+    @classmethod
+    def from_gguf(cls, path: str, max_seq: int = 1024, max_batch: int = 1) -> "Llama":
+        """The model of a GGUF file of architecture "llama" (the file's own tensor names and metadata keys)."""
+        from .gguf import StreamingGGUFReader
+        r = StreamingGGUFReader(path)
+        f = lambda key, default=None: r.fields.get("llama." + key, default)
+        vocab, d_model = r.tensor("token_embd.weight").shape
+        heads = f("attention.head_count")
+        cfg = LlamaConfig(f("block_count"), d_model, heads, f("attention.head_count_kv", heads), f("attention.key_length", d_model // heads),
+                          f("feed_forward_length"), vocab, rms_eps=f("attention.layer_norm_rms_epsilon", 1e-5), rope_theta=f("rope.freq_base", 1e4),
+                          max_seq=max_seq, max_batch=max_batch, linear_enc=r.tensor("blk.0.attn_q.weight").encoding,
+                          table_enc=r.tensor("token_embd.weight").encoding)
+        m = cls(cfg)
+        names = {t.name for t in r.tensors}
+        m.set_weight(0, W_EMBED, r.loadWeightToDevice("token_embd.weight"))
+        m.set_weight(0, W_HEAD, r.loadWeightToDevice("output.weight" if "output.weight" in names else "token_embd.weight"))
+        m.set_norm(0, W_OUT_NORM, r.loadFloats("output_norm.weight"))
+        for l in range(cfg.n_layers):
+            for which, name in ((W_Q, "attn_q"), (W_K, "attn_k"), (W_V, "attn_v"), (W_O, "attn_output"), (W_GATE, "ffn_gate"), (W_UP, "ffn_up"), (W_DOWN, "ffn_down")):
+                m.set_weight(l, which, r.loadWeightToDevice(f"blk.{l}.{name}.weight"))
+            for which, name in ((W_ATTN_NORM, "attn_norm"), (W_FFN_NORM, "ffn_norm")):
+                m.set_norm(l, which, r.loadFloats(f"blk.{l}.{name}.weight"))
+        r.close()
+        m.finalize()
+        return m
 
     # ---- weights --------------------------------------------------------------------------------
     def set_weight(self, layer: int, which: int, w: Weight) -> None:
@@ -94,9 +120,6 @@ class Llama:
         w.free = lambda: None      # borrowed
         return w
 
-    def finalize(self) -> None:
-        L.check(L.lib().skainet_cuda_llama_finalize(self.handle))
-
     @staticmethod
     def tp_unique_id() -> bytes:
         buf = (C.c_uint8 * 128)()
@@ -107,69 +130,9 @@ class Llama:
         buf = (C.c_uint8 * 128).from_buffer_copy(unique_id)
         L.check(L.lib().skainet_cuda_llama_tp_init(self.handle, buf))
 
-    # ---- running ----------------------------------------------------------------------------------
-    def reset(self) -> None:
-        L.check(L.lib().skainet_cuda_llama_reset(self.handle))
-
-    def prefill(self, tokens: Sequence[int], seq: int = 0, want_next: bool = True) -> Optional[int]:
-        t = np.ascontiguousarray(tokens, dtype=np.int32)
-        nxt = C.c_int32(-1)
-        L.check(L.lib().skainet_cuda_llama_prefill(self.handle, seq, t.ctypes.data_as(L.i32p), t.size, C.byref(nxt) if want_next else None))
-        return int(nxt.value) if want_next else None
-
-    def fake_prefill(self, n: int, seq: int = 0, seed: int = 7) -> None:
-        L.check(L.lib().skainet_cuda_llama_fake_prefill(self.handle, seq, n, seed))
-
-    def decode(self, tokens_in: np.ndarray, tokens_out: np.ndarray) -> None:
-        """One greedy step, host tokens in, host tokens out (int32 arrays of length batch; pinned for best latency)."""
-        L.check(L.lib().skainet_cuda_llama_decode(self.handle, tokens_in.size, tokens_in.ctypes.data_as(L.i32p), tokens_out.ctypes.data_as(L.i32p)))
-
-    def decode_ptr(self, batch: int, in_ptr: int, out_ptr: int) -> None:
-        L.check(L.lib().skainet_cuda_llama_decode(self.handle, batch, C.cast(in_ptr, L.i32p), C.cast(out_ptr, L.i32p)))
-
-    def generate(self, first_tokens: Sequence[int], n_steps: int) -> np.ndarray:
-        """n_steps greedy steps on the device; returns [n_steps, batch] tokens."""
-        first = np.ascontiguousarray(first_tokens, dtype=np.int32)
-        out = np.empty((n_steps, first.size), dtype=np.int32)
-        L.check(L.lib().skainet_cuda_llama_generate(self.handle, first.size, first.ctypes.data_as(L.i32p), n_steps, out.ctypes.data_as(L.i32p)))
-        return out
-
-    def logits(self, batch: int = 1) -> np.ndarray:
-        out = np.empty((batch, self.cfg.vocab), dtype=np.float32)
-        L.check(L.lib().skainet_cuda_llama_logits(self.handle, batch, out.ctypes.data_as(L.f32p)))
-        return out
-
-    def peek(self, which: int, n: int) -> np.ndarray:
-        """Diagnostic read of an activation buffer (0 x, 1 q|k|v, 2 attention out, 3 gate|up, 4 q)."""
-        out = np.empty(n, dtype=np.float32)
-        L.check(L.lib().skainet_cuda_llama_peek(self.handle, which, out.ctypes.data_as(L.f32p), n))
-        return out
-
     def tp_exchange_time(self, mode: int, rounds: int = 64, reps: int = 20) -> float:
         """Device microseconds of one group exchange of a [d_model] row, timed on its own (collective: all ranks call it).
         mode 0 peer-memory sum, 1 store + gather + sum + RMSNorm + quantize, 2 NCCL sum."""
         out = C.c_float()
         L.check(L.lib().skainet_cuda_llama_tp_exchange_time(self.handle, mode, rounds, reps, C.byref(out)))
         return float(out.value)
-
-    def step_cost(self, batch: int = 1) -> tuple[int, int]:
-        out = (C.c_int64 * 2)()
-        L.check(L.lib().skainet_cuda_llama_step_cost(self.handle, batch, out))
-        return int(out[0]), int(out[1])
-
-    @property
-    def stream(self) -> int:
-        s = C.c_void_p()
-        L.check(L.lib().skainet_cuda_llama_stream(self.handle, C.byref(s)))
-        return s.value or 0
-
-    def free(self) -> None:
-        if self.handle:
-            L.lib().skainet_cuda_llama_free(self.handle)
-            self.handle = 0
-
-    def __del__(self):
-        try:
-            self.free()
-        except Exception:
-            pass
