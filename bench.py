@@ -30,6 +30,9 @@ Prints ONE JSON line (rank 0). Workloads (all inputs synthetic and seeded):
       in a CUDA graph: the peer-memory sum, the store + gather + sum + RMSNorm + quantize kernel, and ncclAllReduce of the
       same row; metric = microseconds per exchange (lower is better). The N > 1 decode lines carry the same three numbers
       under `tp_exchange`.
+  tivazen — the Tivazen design at --size (7b, 2b, moe: random weights in the shape of a real model's layers) beside a Llama-style
+      Q4_K model of the same layers, width, heads and inner size: greedy decode of --batch sequences behind a --context window
+      and a --prompt-token prefill of each; metric = the Tivazen model's decode tokens/s. One GPU.
   kv_turboquant — the TurboQuant KV store (4-bit keys and values, 8 heads x 128, 32 layers): one decode step of attention over
       --context positions per layer (blocks decoded to fp32, then fp32 attention); metric = microseconds per call (lower is better).
 
@@ -260,6 +263,9 @@ def cpu_attn_rate(workload: str, ctx: int, batch: int) -> dict:
 def run_reference(args) -> None:
     rank, _, _ = dist_env()
     if rank != 0:
+        return
+    if args.workload == "tivazen":
+        print(json.dumps({"impl": "reference", "unavailable": "the reference has no Tivazen model"}), flush=True)
         return
     budget = max(2.0, min(20.0, 90.0 / max(1, args.steps + args.warmup)))
     vals, times = [], []
@@ -869,6 +875,126 @@ def tp_parity_check(torch, dist, m, cfg, model_name: str, ctx: int, batch: int, 
     return out
 
 
+TIVAZEN_SIZES = {
+    # layers, width, heads, kv_rank, window, dense ff, vocab, (experts, top, expert ff) of every second layer or None
+    "7b": (32, 4096, 32, 512, 4096, 11008, 32000, None),
+    "2b": (24, 2048, 16, 512, 1024, 5632, 32000, None),
+    "moe": (24, 2048, 16, 512, 1024, 8448, 102400, (64, 6, 1408)),
+}
+
+
+def tivazen_config(size: str, **kw):
+    """Every second layer reads the cache of the one before it; in "moe" it is routed."""
+    from skainet_b200.tivazen import MLP_DENSE, MLP_MOE, TivazenConfig, TivazenLayer
+    n, width, heads, rank, window, ff, vocab, moe = TIVAZEN_SIZES[size]
+    layers = []
+    for i in range(n):
+        l = TivazenLayer(heads, 128, 64, 128, rank, window, (128 + 64) ** -0.5, 1e4, i - 1 if i % 2 else None, MLP_DENSE, ff)
+        if moe and i % 2:
+            l.mlp, (l.experts, l.top, l.ff) = MLP_MOE, moe
+        layers.append(l)
+    return TivazenConfig(width, vocab, 1e-5, layers, **kw)
+
+
+def tivazen_linear_flops(cfg) -> float:
+    """Multiply-adds x 2 of the linears per prompt token (the attention over the cache comes on top)."""
+    total = 0
+    for l in cfg.layers:
+        own = l.kv_from is None
+        total += cfg.width * (l.heads * (l.dim + l.rot_dim) + (l.kv_rank + l.rot_dim if own else 0) + l.heads + l.experts)
+        total += l.heads * l.kv_rank * (l.dim + l.vdim) + cfg.width * l.heads * l.vdim + 3 * cfg.width * l.ff * (l.top or 1)
+    return 2.0 * total
+
+
+def decoder_phases(torch, m, batch: int, ctx: int, n_prompt: int, steps: int, warm: int, vocab: int) -> dict:
+    """Decode of `batch` sequences behind ctx noise tokens, and the prefill of one n_prompt-token prompt, device time."""
+    mstream = torch.cuda.ExternalStream(m.stream)
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+    first = np.arange(1, batch + 1, dtype=np.int32)
+
+    def context():
+        m.reset()
+        for b in range(batch):
+            m.fake_prefill(ctx, b)
+    context()
+    bytes_step, launches = m.step_cost(batch)
+    m.generate(first, warm)
+    best = []
+    for _ in range(3):
+        context()
+        m.generate(first, 1)
+        a, b = ev(), ev()
+        a.record(mstream); m.generate(first, steps); b.record(mstream)
+        torch.cuda.synchronize()
+        best.append(a.elapsed_time(b) / steps)
+    ms = float(np.median(best))
+    context()
+    tin = torch.from_numpy(first.copy()).pin_memory(); tout = torch.zeros(batch, dtype=torch.int32).pin_memory()
+    t0 = time.perf_counter()
+    for _ in range(steps):
+        m.decode_ptr(batch, tin.data_ptr(), tout.data_ptr()); tin.copy_(tout)
+    e2e = (time.perf_counter() - t0) * 1e3 / steps
+    prompt = np.random.default_rng(11).integers(0, vocab, n_prompt).astype(np.int32)
+    pre = []
+    for i in range(warm + 5):
+        m.reset()
+        a, b = ev(), ev()
+        a.record(mstream); m.prefill(prompt, 0, want_next=False); b.record(mstream)
+        torch.cuda.synchronize()
+        if i >= warm:
+            pre.append(a.elapsed_time(b))
+    return {"decode_ms": ms, "decode_tokens_per_s": batch / ms * 1e3, "e2e_ms": e2e, "bytes_per_step": bytes_step, "launches_per_step": launches,
+            "decode_gbs": bytes_step / ms / 1e6, "prefill_ms": float(np.median(pre)), "prefill_tokens_per_s": n_prompt / float(np.median(pre)) * 1e3}
+
+
+def run_tivazen(args) -> None:
+    import torch
+    from skainet_b200 import _lib as L, device
+    from skainet_b200.llama import Llama, LlamaConfig
+    from skainet_b200.tivazen import Tivazen
+    rank, world, local = dist_env()
+    torch.cuda.set_device(local); device.set_device(local)
+    n, width, heads, rank_kv, window, ff, vocab, moe = TIVAZEN_SIZES[args.size]
+    batch, ctx, n_prompt, warm = max(1, args.batch), min(args.context, window), args.prompt, max(3, args.warmup)
+    room = max(ctx + args.steps + warm + 8, n_prompt)
+    sampler = ClockSampler(local); sampler.start()
+    cfg = tivazen_config(args.size, max_seq=room, max_batch=batch)
+    m = Tivazen(cfg)
+    m.synth(seed=100, std=0.02)
+    m.finalize()
+    ours = decoder_phases(torch, m, batch, ctx, n_prompt, args.steps, warm, vocab)
+    m.free()
+    near = None
+    if not args.skip_cpu:
+        k = Llama(LlamaConfig(n, width, heads, heads, 128, ff, vocab, max_seq=room, max_batch=batch))
+        k.synth(seed=100, std=0.02)
+        k.finalize()
+        near = decoder_phases(torch, k, batch, ctx, n_prompt, args.steps, warm, vocab)
+        k.free()
+    clocks = sampler.stop()
+    if L.lib().skainet_cuda_device_status() != 0:
+        raise SystemExit(f"device error: {L.last_error()}")
+    peak, peak_kind = load_peaks()
+    tpeak, _ = load_tensor_peak()
+    ours["prefill_linear_tflops"] = tivazen_linear_flops(cfg) * n_prompt / ours["prefill_ms"] / 1e9
+    ours["prefill_frac_of_bf16_burst"] = ours["prefill_linear_tflops"] / tpeak
+    if near:
+        near["prefill_linear_tflops"] = 2.0 * n * (4 * width * width + 3 * width * ff) * n_prompt / near["prefill_ms"] / 1e9
+        near["prefill_frac_of_bf16_burst"] = near["prefill_linear_tflops"] / tpeak
+        near["decode_frac"] = near["decode_gbs"] / peak
+    line = {"metric": "tivazen_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": warm,
+            "ms_per_step": ours["decode_ms"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+            "dtype": "bf16 weights, activations and cache, f32 accumulate (residual, norms, scores, routing f32)", "data": "synthetic",
+            "config": {"workload": "tivazen", "size": args.size, "layers": n, "width": width, "heads": heads, "kv_rank": rank_kv, "window": window, "ff": ff, "vocab": vocab,
+                       "routed": moe, "batch": batch, "context": ctx, "context_fill": "seeded noise", "prompt_tokens": n_prompt, "weights": "N(0,0.02), seeded",
+                       "l2": "weights per step far larger than L2", "parallelism": "single"},
+            "roofline": {"bound": "hbm", "achieved": ours["decode_gbs"], "peak": peak, "unit": "GB/s", "frac": ours["decode_gbs"] / peak, "traffic": None,
+                         "peak_kind": peak_kind, "kernel": "whole decode step"},
+            "tivazen": ours, "closest_llama_q4k": near, "gpu_launches": ours["launches_per_step"] * args.steps, "clocks": clocks,
+            "e2e": {"value": batch / ours["e2e_ms"] * 1e3, "unit": "tokens/s", "h2d_bytes_per_step": 4 * batch, "d2h_bytes_per_step": 4 * batch}}
+    print(json.dumps(line), flush=True)
+
+
 def run_kv_turboquant(args) -> None:
     """kv_turboquant: the TurboQuant KV store (4-bit keys and values, 8 heads x 128) behind one decode step of attention over
     --context positions: decode of the window's blocks to fp32 + fp32 attention, per layer of a 32-layer store (the layers'
@@ -1156,11 +1282,13 @@ def main() -> None:
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=5)
-    ap.add_argument("--workload", default="decode_70b", choices=sorted(MATVEC_WORKLOADS) + sorted(DECODE_WORKLOADS) + sorted(ATTN_WORKLOADS) + sorted(GEMM_WORKLOADS) + sorted(REQUEST_WORKLOADS) + ["tp_collective", "kv_turboquant"])
-    ap.add_argument("--context", type=int, default=4096, help="keys per sequence (attn_decode workload)")
+    ap.add_argument("--workload", default="decode_70b", choices=sorted(MATVEC_WORKLOADS) + sorted(DECODE_WORKLOADS) + sorted(ATTN_WORKLOADS) + sorted(GEMM_WORKLOADS) + sorted(REQUEST_WORKLOADS) + ["tivazen", "tp_collective", "kv_turboquant"])
+    ap.add_argument("--context", type=int, default=4096, help="keys per sequence (attn_decode, tivazen workloads)")
     ap.add_argument("--batch", type=int, default=1, help="sequences decoded together (decode workloads)")
+    ap.add_argument("--size", default="7b", choices=sorted(TIVAZEN_SIZES), help="model shape of the tivazen workload")
+    ap.add_argument("--prompt", type=int, default=2048, help="prompt tokens of the tivazen workload's prefill")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--skip-cpu", action="store_true", help="omit the cpu_baseline leg (profiling runs)")
+    ap.add_argument("--skip-cpu", action="store_true", help="omit the cpu_baseline leg, or the Llama-style comparison of the tivazen workload (profiling runs)")
     ap.add_argument("--skip-e2e", action="store_true", help="omit the end-to-end leg (profiling runs)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -1175,6 +1303,8 @@ def main() -> None:
         run_request(args)
     elif args.workload == "tp_collective":
         run_collective(args)
+    elif args.workload == "tivazen":
+        run_tivazen(args)
     elif args.workload == "kv_turboquant":
         run_kv_turboquant(args)
     else:

@@ -1,5 +1,5 @@
 """Plain restatement of a Tivazen decoder in numpy double precision: one function per mechanism, whole sequences at once,
-no cache and no batching. It is the checker of tests/test_tivazen*.py and shares no code with the product path.
+no cache and no batching. It is the oracle of the tests of that design and shares no code with the product path.
 
 A model is `cfg` (the parsed config.json) and `w`, a dict of float arrays under the names of model.safetensors."""
 from __future__ import annotations
