@@ -12,12 +12,10 @@
 // whose product silu(gate) * up is then formed in the epilogue without a round trip.
 // Every mbarrier wait is bounded; a wait that runs out raises the device flag and the CTA still frees its TMEM.
 #include "linear_bf16.cuh"
+#include "tensor_map.cuh"
 #include "tma.cuh"
 
-#include <cuda.h>
-
 #include <algorithm>
-#include <mutex>
 
 namespace sk {
 
@@ -61,10 +59,6 @@ __device__ __forceinline__ void umma_commit(uint64_t* bar) {
 }
 __device__ __forceinline__ void arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(skd::smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tma_tile(void* dst, const CUtensorMap* map, int k, int row, uint64_t* bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-                 ::"r"(skd::smem_u32(dst)), "l"(map), "r"(k), "r"(row), "r"(skd::smem_u32(bar)) : "memory");
 }
 __device__ __forceinline__ void tmem_ld32(uint32_t ta, float (&u)[32]) {
     uint32_t r[32];
@@ -145,9 +139,9 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 if (it >= S::STAGES && !(ok = skd::mbar_wait_bounded(empty + s, ((it / S::STAGES) + 1) & 1, a.timeout_flag))) break;
                 uint8_t* st = smem + s * S::STAGE;
                 skd::mbar_expect_tx(full + s, S::STAGE);
-                tma_tile(st, &map_a, k * BKE, wrow, full + s);
-                if (NA == 2) tma_tile(st + A_BYTES, &map_a2, k * BKE, wrow + a.a2_rows, full + s);
-                tma_tile(st + NA * A_BYTES, &map_b, xk + k * BKE, tl.x_row, full + s);
+                skd::tma_load_2d(st, &map_a, k * BKE, wrow, full + s);
+                if (NA == 2) skd::tma_load_2d(st + A_BYTES, &map_a2, k * BKE, wrow + a.a2_rows, full + s);
+                skd::tma_load_2d(st + NA * A_BYTES, &map_b, xk + k * BKE, tl.x_row, full + s);
             }
         }
         // copies still in flight must land before the CTA leaves: the last round of each posted stage
@@ -220,39 +214,14 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(S::TMEM) : "memory");
 }
 
-typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
-                             const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeFn encode_fn() {
-    static EncodeFn fn = [] {
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) { cudaGetLastError(); p = nullptr; }
-        return (EncodeFn) p;
-    }();
-    return fn;
-}
-
-// [rows][ld] bf16, boxes of `box_rows` x 64 elements in the 128-byte swizzle; rows outside read as zero.
-int32_t make_map(CUtensorMap* map, const bf16* base, int64_t rows, int ld, int box_rows) {
-    EncodeFn fn = encode_fn();
-    SK_REQUIRE(fn != nullptr, "gemm_bf16_tc: the driver has no tensor-map encoder");
-    const cuuint64_t dims[2] = {(cuuint64_t) ld, (cuuint64_t) rows};
-    const cuuint64_t strides[1] = {(cuuint64_t) ld * 2};
-    const cuuint32_t box[2] = {BKE, (cuuint32_t) box_rows}, es[2] = {1, 1};
-    const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(base), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                          CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    SK_REQUIRE(r == CUDA_SUCCESS, "gemm_bf16_tc: tensor map of [%lld, %d] refused (%d)", (long long) rows, ld, (int) r);
-    return SKAINET_CUDA_OK;
-}
-
 template <int NA, int BN, int OUT>
 int32_t run_tc(const LinearArgs& l, cudaStream_t s) {
     typedef Shape<NA, BN> S;
     CUtensorMap ma, ma2, mb;
     const int64_t w_total = (int64_t) l.groups * l.w_rows;
-    SK_TRY(make_map(&ma, l.w, w_total, l.ldw, BM));
-    if (OUT == LIN_OUT_SWIGLU) SK_TRY(make_map(&ma2, l.w2, w_total, l.ldw, BM)); else ma2 = ma;
-    SK_TRY(make_map(&mb, (const bf16*) l.x, l.x_rows_alloc, l.ldx, BN));
+    SK_TRY(tensor_map_rows(&ma, l.w, w_total, l.ldw, BM));
+    if (OUT == LIN_OUT_SWIGLU) SK_TRY(tensor_map_rows(&ma2, l.w2, w_total, l.ldw, BM)); else ma2 = ma;
+    SK_TRY(tensor_map_rows(&mb, (const bf16*) l.x, l.x_rows_alloc, l.ldx, BN));
     TcArgs a = {};
     a.y = l.y; a.ldy = l.ldy; a.y_group_stride = l.y_group_stride; a.scale = l.scale; a.scale_ld = l.scale_ld;
     a.segs = l.segs; a.n_segs = l.n_segs; a.w_rows = l.w_rows; a.rows = l.rows; a.groups = l.groups;

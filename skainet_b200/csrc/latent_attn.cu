@@ -89,20 +89,47 @@ __device__ __forceinline__ float dot8(uint4 w, const float* x) {
            skd::bf16_lo(w.z) * x[4] + skd::bf16_hi(w.z) * x[5] + skd::bf16_lo(w.w) * x[6] + skd::bf16_hi(w.w) * x[7];
 }
 
-// y[o] = sum_k W[o][k] x[k] for output rows o0 <= o < o1 by a CTA of 256 threads: `lanes` (8, 16 or 32) threads per row.
-template <typename F>
-__device__ __forceinline__ void cta_matvec(const bf16* w, int ld, const float* x, int o0, int o1, F&& store) {
-    const int lanes = ld >= 256 ? 32 : (ld >= 128 ? 16 : 8), per = 256 / lanes;
-    const int l = threadIdx.x % lanes, r = threadIdx.x / lanes;
-    for (int b = o0; b < o1; b += per) {
-        const int o = b + r;
-        float v = 0.0f;
-        if (o < o1)
-            for (int k = l * 8; k < ld; k += lanes * 8) v += dot8(skd::ld_ro(w + (size_t) o * ld + k), x + k);
-        for (int m = lanes / 2; m > 0; m >>= 1) v += __shfl_xor_sync(~0u, v, m);
-        if (l == 0 && o < o1) store(o, v);
+// y[o] = sum_k W[o][k] x[k] for output rows o0 <= o < o1 by a CTA of 256 threads: `lanes` (8, 16 or 32) threads per row. The
+// first AHEAD loads of every thread are issued by the constructor, which needs no input from the preceding kernel.
+constexpr int AHEAD = 8;
+struct CtaMatvec {
+    const bf16* w;
+    int ld, lanes, l, r, per, o0, o1, nk, total;
+    uint4 pre[AHEAD];
+    __device__ __forceinline__ uint4 load(int i) const {
+        const int o = o0 + (i / nk) * per + r, k = (i % nk) * lanes * 8 + l * 8;
+        return i < total && o < o1 && k < ld ? skd::ld_ro(w + (size_t) o * ld + k) : make_uint4(0, 0, 0, 0);
     }
-}
+    __device__ __forceinline__ CtaMatvec(const bf16* w_, int ld_, int o0_, int o1_) : w(w_), ld(ld_), o0(o0_), o1(o1_) {
+        lanes = ld >= 256 ? 32 : (ld >= 128 ? 16 : 8); per = 256 / lanes;
+        l = threadIdx.x % lanes; r = threadIdx.x / lanes;
+        nk = (ld + lanes * 8 - 1) / (lanes * 8);
+        total = o1 > o0 ? (o1 - o0 + per - 1) / per * nk : 0;
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) pre[i] = load(i);
+    }
+    template <typename F>
+    __device__ __forceinline__ void run(const float* x, F&& store) {
+        float v = 0.0f;
+        for (int i0 = 0; i0 < total; i0 += AHEAD) {
+            if (i0 > 0) {
+#pragma unroll
+                for (int i = 0; i < AHEAD; ++i) pre[i] = load(i0 + i);
+            }
+#pragma unroll
+            for (int i = 0; i < AHEAD; ++i) {
+                if (i0 + i >= total) break;
+                const int kb = (i0 + i) % nk, o = o0 + (i0 + i) / nk * per + r, k = kb * lanes * 8 + l * 8;
+                if (k < ld) v += dot8(pre[i], x + k);
+                if (kb == nk - 1) {
+                    for (int m = lanes / 2; m > 0; m >>= 1) v += __shfl_xor_sync(~0u, v, m);
+                    if (l == 0 && o < o1) store(o, v);
+                    v = 0.0f;
+                }
+            }
+        }
+    }
+};
 
 // Few rows: grid (heads + 1, rows, parts). Head CTAs rotate their query and fold a part of W_uk into it; the last column
 // prepares latent, key part and gates.
@@ -110,24 +137,25 @@ __global__ void __launch_bounds__(256) latent_prep_fold_kernel(const LatentArgs 
     extern __shared__ float sq[];
     __shared__ float sh[8];
     skd::pdl_launch_dependents();
-    skd::pdl_wait();
     const LatentGeom& g = a.g;
     const int h = blockIdx.x, row = blockIdx.y;
     if (h == g.heads) {
+        skd::pdl_wait();
         if (blockIdx.z == 0) prep_row<bf16>(a, row, sh);
         return;
     }
+    const int ld = g.dim_ld(), per = (g.kv_rank + gridDim.z - 1) / gridDim.z, o0 = blockIdx.z * per;
+    CtaMatvec mv(a.uk_t + (size_t) h * g.kv_rank * ld, ld, o0, min(g.kv_rank, o0 + per));
+    skd::pdl_wait();
     const float* q = a.proj + (size_t) row * a.proj_ld + (size_t) h * (g.dim + g.rot_dim);
-    const int ld = g.dim_ld();
     for (int i = threadIdx.x; i < ld; i += 256) sq[i] = i < g.dim ? q[i] : 0.0f;
     if (blockIdx.z == 0) {
         const int pos = a.map.pos_of(row);
         for (int i = threadIdx.x; i < (g.rot_dim >> 1); i += 256) rotate_query<bf16>(a, row, h, i, pos);
     }
     __syncthreads();
-    const int per = (g.kv_rank + gridDim.z - 1) / gridDim.z, o0 = blockIdx.z * per, o1 = min(g.kv_rank, o0 + per);
     bf16* dst = (bf16*) a.qf + ((size_t) row * g.heads + h) * g.key_ld();
-    cta_matvec(a.uk_t + (size_t) h * g.kv_rank * ld, ld, sq, o0, o1, [&](int o, float v) { dst[o] = __float2bfloat16_rn(v); });
+    mv.run(sq, [&](int o, float v) { dst[o] = __float2bfloat16_rn(v); });
 }
 
 // ---- attention over the cache ---------------------------------------------------------------------------------------
@@ -179,13 +207,6 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
     const int t0 = split * per, t1 = min(n_tiles, t0 + per);
     const bf16* cache = (const bf16*) a.cache.rows + (size_t) seq * a.cache.cap * kld;
 
-    for (int m = warp; m < ROWS; m += 8) {                    // query rows, zero where there is none
-        const int r = r0 + m / hb, h = h0 + m % hb;
-        const bool live = m < sp.rows_per_block * hb && r <= r_last && h < g.heads;
-        if (lane == 0) qpos[m] = live ? a.map.pos_of(r) : -1;
-        const uint4* src = (const uint4*) ((const bf16*) a.qf + ((size_t) (live ? r : 0) * g.heads + (live ? h : 0)) * kld);
-        for (int c = lane; c < chunks; c += 32) *(uint4*) (sq + m * sld + c * 8) = live ? src[c] : make_uint4(0, 0, 0, 0);
-    }
     auto fetch = [&](int t) {                                 // keys past hi repeat the newest one; their weights are masked
         if (t < t1) {
             bf16* dst = sk_ + (t % ST) * BK * sld;
@@ -198,6 +219,13 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     for (int i = 0; i < ST - 1; ++i) fetch(t0 + i);
+    for (int m = warp; m < ROWS; m += 8) {                    // query rows, zero where there is none
+        const int r = r0 + m / hb, h = h0 + m % hb;
+        const bool live = m < sp.rows_per_block * hb && r <= r_last && h < g.heads;
+        if (lane == 0) qpos[m] = live ? a.map.pos_of(r) : -1;
+        const uint4* src = (const uint4*) ((const bf16*) a.qf + ((size_t) (live ? r : 0) * g.heads + (live ? h : 0)) * kld);
+        for (int c = lane; c < chunks; c += 32) *(uint4*) (sq + m * sld + c * 8) = live ? src[c] : make_uint4(0, 0, 0, 0);
+    }
 
     float acc[NT][2][4];
 #pragma unroll
@@ -233,20 +261,28 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
             }
         } else {
             const bf16* bk = kt + (nw * 8 + (lane & 7)) * sld + (lane >> 3) * 8;
+            float s1[4] = {}, s2[4] = {}, s3[4] = {};         // four independent accumulator chains
             int k = 0;
-            for (; k + 32 <= kld; k += 32) {
-                uint32_t fa[4], fc[4], fb[4];
-                ldsm4(fb, bk + k); ldsm4(fa, aq + k); ldsm4(fc, aq + k + 16);
+            for (; k + 64 <= kld; k += 64) {
+                uint32_t fa[4], fb[4];
+                ldsm4(fb, bk + k); ldsm4(fa, aq + k);
                 skd::mma_bf16(s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
-                skd::mma_bf16(s4[0], fc[0], fc[1], fc[2], fc[3], fb[2], fb[3]);
+                ldsm4(fa, aq + k + 16);
+                skd::mma_bf16(s1, fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
+                ldsm4(fb, bk + k + 32); ldsm4(fa, aq + k + 32);
+                skd::mma_bf16(s2, fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
+                ldsm4(fa, aq + k + 48);
+                skd::mma_bf16(s3, fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
             }
-            if (k < kld) {                                    // odd number of k16 steps: the upper half of the load falls in the row's padding or the next row, unused
+            for (; k < kld; k += 16) {
                 uint32_t fa[4], fb[2];
                 ldsm4(fa, aq + k);
                 asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(fb[0]), "=r"(fb[1])
                              : "r"(skd::smem_u32(kt + (nw * 8 + (lane & 7)) * sld + ((lane >> 3) & 1) * 8 + k)) : "memory");
                 skd::mma_bf16(s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
             }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) s4[0][j] += s1[j] + (s2[j] + s3[j]);
         }
         // scaled scores in powers of two, masked; row maxima over this warp's keys, then over the warps
         const int pa = qpos[ra], pb = qpos[rb];
@@ -397,51 +433,75 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(const LatentArgs 
 }
 
 // ---- key splits -----------------------------------------------------------------------------------------------------
-// The mixed latent of (row, head) from its split records, columns strided over the CTA, handed to store(c, value).
+// The mixed latent of (row, head) from its split records by a CTA of 256 threads, handed to store(column, value). The factors
+// of the splits are formed once; then groups of threads take every n-th split of four columns and meet in shared memory.
+constexpr int MERGE_MAX_SPLITS = 256;
 template <typename F>
-__device__ __forceinline__ void merge_splits(const float* part, int n_splits, int RP, F&& store) {
-    float m = NEG_BIG, l = 0.0f;
-    for (int s = 0; s < n_splits; ++s) if (part[(size_t) s * (RP + 2) + RP + 1] > 0.0f) m = fmaxf(m, part[(size_t) s * (RP + 2) + RP]);
-    for (int s = 0; s < n_splits; ++s) {
-        const float* d = part + (size_t) s * (RP + 2) + RP;
-        if (d[1] > 0.0f) l += d[1] * exp2f(d[0] - m);
+__device__ __forceinline__ void merge_splits(const float* part, int n_splits, int RP, float* fac, float4* sums, F&& store) {
+    const int rec = RP + 2;
+    float m = NEG_BIG;
+    for (int s = threadIdx.x & 31; s < n_splits; s += 32) if (part[(size_t) s * rec + RP + 1] > 0.0f) m = fmaxf(m, part[(size_t) s * rec + RP]);
+    m = skd::warp_max(m);
+    float l = 0.0f;
+    for (int s = threadIdx.x & 31; s < n_splits; s += 32) {
+        const float ls = part[(size_t) s * rec + RP + 1], f = ls > 0.0f ? exp2f(part[(size_t) s * rec + RP] - m) : 0.0f;
+        l += ls * f;
+        if (threadIdx.x < 32) fac[s] = f;
     }
-    const float inv = 1.0f / l;
-    for (int c = threadIdx.x; c < RP; c += blockDim.x) {
-        float v = 0.0f;
-        for (int s = 0; s < n_splits; ++s) {
-            const float* d = part + (size_t) s * (RP + 2);
-            if (d[RP + 1] > 0.0f) v = fmaf(d[c], exp2f(d[RP] - m), v);      // a split that held no visible key wrote no usable sums
+    const float inv = 1.0f / skd::warp_sum(l);
+    __syncthreads();
+    const int q4 = RP / 4;                                  // column quads; RP is a multiple of 16
+    for (int c0 = 0; c0 < q4; c0 += 256) {
+        const int cols = min(256, q4 - c0), ways = 256 / cols, c = threadIdx.x % cols, w = threadIdx.x / cols;
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (w < ways) {
+#pragma unroll 8
+            for (int s = w; s < n_splits; s += ways) {
+                const float f = fac[s];
+                const float2* d = reinterpret_cast<const float2*>(part + (size_t) s * rec + 4 * (c0 + c));
+                const float2 a = d[0], b = d[1];
+                v.x = fmaf(a.x, f, v.x); v.y = fmaf(a.y, f, v.y); v.z = fmaf(b.x, f, v.z); v.w = fmaf(b.y, f, v.w);
+            }
+            sums[threadIdx.x] = v;
         }
-        store(c, v * inv);
+        __syncthreads();
+        if ((int) threadIdx.x < cols) {
+            for (int k = 1; k < ways; ++k) { const float4 o = sums[k * cols + c]; v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w; }
+            const int at = 4 * (c0 + c);
+            store(at, v.x * inv); store(at + 1, v.y * inv); store(at + 2, v.z * inv); store(at + 3, v.w * inv);
+        }
+        __syncthreads();
     }
 }
 
 template <typename T>
-__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentArgs a, int n_splits) {
+__global__ void __launch_bounds__(256) latent_merge_kernel(const LatentArgs a, int n_splits) {
+    __shared__ float fac[MERGE_MAX_SPLITS];
+    __shared__ float4 sums[256];
     skd::pdl_launch_dependents();
     skd::pdl_wait();
     const LatentGeom& g = a.g;
     const size_t rh = (size_t) blockIdx.y * g.heads + blockIdx.x;
     T* d = (T*) a.mix + rh * g.rank_ld();
-    merge_splits(a.part + rh * n_splits * (g.rank_pad() + 2), n_splits, g.rank_pad(), [&](int c, float v) { skd::store_act(d + c, v); });
+    merge_splits(a.part + rh * n_splits * (g.rank_pad() + 2), n_splits, g.rank_pad(), fac, sums, [&](int c, float v) { skd::store_act(d + c, v); });
 }
 
 // Few rows: grid (heads, rows, parts): merge, then a part of W_uv's rows, gated.
 __global__ void __launch_bounds__(256) latent_merge_value_kernel(const LatentArgs a, int n_splits) {
     extern __shared__ float so[];
+    __shared__ float fac[MERGE_MAX_SPLITS];
+    __shared__ float4 sums[256];
     skd::pdl_launch_dependents();
-    skd::pdl_wait();
     const LatentGeom& g = a.g;
-    const int h = blockIdx.x, row = blockIdx.y, ld = g.rank_ld();
+    const int h = blockIdx.x, row = blockIdx.y, ld = g.rank_ld(), per = (g.vdim + gridDim.z - 1) / gridDim.z, o0 = blockIdx.z * per;
+    CtaMatvec mv(a.uv + (size_t) h * g.vdim * ld, ld, o0, min(g.vdim, o0 + per));
+    skd::pdl_wait();
     const size_t rh = (size_t) row * g.heads + h;
     for (int i = g.rank_pad() + threadIdx.x; i < ld; i += 256) so[i] = 0.0f;
-    merge_splits(a.part + rh * n_splits * (g.rank_pad() + 2), n_splits, g.rank_pad(), [&](int c, float v) { so[c] = v; });
-    __syncthreads();
+    merge_splits(a.part + rh * n_splits * (g.rank_pad() + 2), n_splits, g.rank_pad(), fac, sums, [&](int c, float v) { so[c] = v; });
     const float gate = a.gates[rh];
     bf16* dst = (bf16*) a.out + (size_t) row * g.out_ld() + (size_t) h * g.vdim;
-    const int per = (g.vdim + gridDim.z - 1) / gridDim.z, o0 = blockIdx.z * per, o1 = min(g.vdim, o0 + per);
-    cta_matvec(a.uv + (size_t) h * g.vdim * ld, ld, so, o0, o1, [&](int o, float v) { dst[o] = __float2bfloat16_rn(v * gate); });
+    mv.run(so, [&](int o, float v) { dst[o] = __float2bfloat16_rn(v * gate); });
 }
 
 __global__ void transpose_heads_kernel(const bf16* __restrict__ src, bf16* __restrict__ dst, int dim, int kv_rank, int src_ld, int dst_ld) {
@@ -512,7 +572,7 @@ int32_t launch_latent_attention(const LatentArgs& args, cudaStream_t s) {
     } else grid = dim3(1, g.heads, a.rows);
     const int64_t blocks = (int64_t) grid.y * grid.z, records = (int64_t) a.rows * g.heads;
     const int keys = std::min(a.kv_bound, a.window + sp.rows_per_block - 1), tiles = (keys + bk - 1) / bk;
-    sp.n_splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) sm_count() / std::max<int64_t>(1, blocks), (int64_t) tiles, LATENT_PART_RECORDS / std::max<int64_t>(1, records)}));
+    sp.n_splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) sm_count() / std::max<int64_t>(1, blocks), (int64_t) (tiles + 1) / 2, MERGE_MAX_SPLITS, LATENT_PART_RECORDS / std::max<int64_t>(1, records)}));
     grid.x = sp.n_splits;
     if (!few && sp.n_splits == 1) a.part = nullptr;
     if (mma) SK_TRY(launch_mma(a, sp, mw, grid, s));
@@ -532,8 +592,8 @@ int32_t launch_latent_attention(const LatentArgs& args, cudaStream_t s) {
         return SKAINET_CUDA_OK;
     }
     if (a.part) {
-        if (a.f32_act) SK_CUDA(launch_pdl(latent_merge_kernel<float>, dim3(g.heads, a.rows), dim3(128), 0, s, a, sp.n_splits));
-        else SK_CUDA(launch_pdl(latent_merge_kernel<bf16>, dim3(g.heads, a.rows), dim3(128), 0, s, a, sp.n_splits));
+        if (a.f32_act) SK_CUDA(launch_pdl(latent_merge_kernel<float>, dim3(g.heads, a.rows), dim3(256), 0, s, a, sp.n_splits));
+        else SK_CUDA(launch_pdl(latent_merge_kernel<bf16>, dim3(g.heads, a.rows), dim3(256), 0, s, a, sp.n_splits));
     }
     LinearArgs l;
     l.w = a.uv; l.w_rows = g.vdim; l.ldw = g.rank_ld(); l.groups = g.heads; l.x = a.mix; l.ldx = g.heads * g.rank_ld(); l.x_group_stride = g.rank_ld();

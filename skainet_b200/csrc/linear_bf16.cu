@@ -1,12 +1,13 @@
 // Linears over BF16 weights (contract: linear_bf16.cuh).
 //
-//   linear_skinny_kernel  up to 16 activation rows (decode): every weight byte is read once, straight from HBM into the
-//                         mma.sync A fragments; bound by the weight stream, the tensor instructions only save the CUDA
-//                         cores the unpacking. K is permuted identically in both operands so that a lane's 16-byte load
+//   linear_ring_kernel    up to 16 activation rows (decode): every weight byte is read once, through a ring of shared-memory
+//                         stages filled by TMA; bound by the weight stream. The arithmetic is mma.sync: it only saves the CUDA
+//                         cores the unpacking. K is permuted identically in both operands, so that a lane's 16-byte load
 //                         (8 consecutive k of a row) is two k16 steps' worth of its A fragment.
 //   linear_f32_kernel     fp32 activations, fp32 FMA: the 32-bit mode, every row count.
 //   gemm_bf16_tc.cu       more rows: tcgen05.
 #include "linear_bf16.cuh"
+#include "tensor_map.cuh"
 #include "tma.cuh"
 
 #include <algorithm>
@@ -15,106 +16,154 @@ namespace sk {
 
 namespace {
 
-constexpr int SK_WARPS = 8, SK_TILE = 16;
+constexpr int RG_WARPS = 8, RG_TILE = 16, RG_THREADS = (RG_WARPS + 1) * 32;
+constexpr int RG_SMEM = 96 * 1024;       // ring and partial sums of two CTAs fit an SM
 
-// CTA = 16 output rows of one group (or one segment's expert); its eight warps take every eighth k32 step, then the partial
-// sums meet in shared memory in fixed order. NB = tiles of 8 activation rows.
-template <int NB, int OUT, int U>
-__global__ void __launch_bounds__(SK_WARPS * 32)
-linear_skinny_kernel(const LinearArgs a) {
+// MT weight matrices (gate and up), 16 rows of each per unit; a stage holds KB blocks of 64 k: [matrix][block][16 rows][128 bytes],
+// the 16-byte chunks of a row XORed with the row (the copy engine's 128-byte swizzle). One copy instruction per matrix and stage:
+// with one per row the stream was bound by the issue of the copies (1.9-3.2 TB/s).
+template <int MT>
+struct Ring {
+    static constexpr int KB = MT == 1 ? 8 : 4, KC = KB * 64, MAT = KB * RG_TILE * 128, STAGE = MT * MAT;
+    static constexpr int STAGES = (RG_SMEM - (MT - 1) * 16 * 1024) / STAGE;
+};
+template <int MT, int NB>
+constexpr int ring_smem() { return Ring<MT>::STAGES * Ring<MT>::STAGE + 2 * RG_WARPS * MT * NB * RG_TILE * 8 * 4 + 2 * Ring<MT>::STAGES * 8 + 1024; }
+
+// Persistent CTA; a unit is 16 output rows of one group (or of one segment's expert) over all of K. One producer warp streams
+// the units' rows; eight consumer warps take every eighth k32 step of a stage, and their partial sums meet in shared memory in
+// fixed order at the end of a unit. NB = tiles of 8 activation rows.
+template <int NB, int OUT>
+__global__ void __launch_bounds__(RG_THREADS, 2)
+linear_ring_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_w2, const LinearArgs a, int* __restrict__ timeout_flag) {
     constexpr bool DUAL = OUT == LIN_OUT_SWIGLU;
     constexpr int MT = DUAL ? 2 : 1;
-    __shared__ float part[SK_WARPS][MT][NB][SK_TILE * 8 + 4];
-    skd::pdl_launch_dependents();
+    typedef Ring<MT> R;
+    extern __shared__ uint8_t raw[];
+    uint8_t* smem = raw + ((1024 - (skd::smem_u32(raw) & 1023)) & 1023);
+    float* part = (float*) (smem + R::STAGES * R::STAGE);               // [2][warps][MT][NB][8 * 16]
+    uint64_t* full = (uint64_t*) (part + 2 * RG_WARPS * MT * NB * RG_TILE * 8);
+    uint64_t* empty = full + R::STAGES;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    const int tile = blockIdx.x * SK_TILE;
-    const int steps = a.ldw >> 5;
-    int group = blockIdx.y, row0 = 0, n_rows = a.rows;
-    if (a.segs) {
-        skd::pdl_wait();
-        if ((int) blockIdx.y >= *a.n_segs) return;
-        const RowSegment sg = a.segs[blockIdx.y];
-        group = sg.group; row0 = sg.start; n_rows = sg.count;
+    skd::pdl_launch_dependents();
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < R::STAGES; ++s) { skd::mbar_init(full + s, 1); skd::mbar_init(empty + s, RG_WARPS); }
+        skd::mbar_fence_init();
     }
-    const size_t goff = (size_t) group * a.w_rows * a.ldw;
-    const bf16* wp[MT][2];
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-        const size_t off = goff + (size_t) min(tile + g + 8 * h, a.w_rows - 1) * a.ldw + 8 * t;
-        wp[0][h] = a.w + off;
-        if (DUAL) wp[MT - 1][h] = a.w2 + off;
-    }
-    uint4 wr[U][MT][2];
-    auto load_w = [&](int st0) {
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int st = st0 + u * SK_WARPS;
-#pragma unroll
-            for (int m = 0; m < MT; ++m)
-#pragma unroll
-                for (int h = 0; h < 2; ++h) wr[u][m][h] = st < steps ? skd::ld_stream(wp[m][h] + (size_t) st * 32) : make_uint4(0, 0, 0, 0);
-        }
-    };
-    load_w(warp);                            // weights do not depend on the predecessor: in flight before the wait
-    if (!a.segs) skd::pdl_wait();
-    const bf16* xp[NB];
-    bool live[NB];
-#pragma unroll
-    for (int b = 0; b < NB; ++b) {
-        const int n = b * 8 + g;
-        live[b] = n < n_rows;
-        const int r = live[b] ? (a.row_index ? a.row_index[row0 + n] : row0 + n) : 0;
-        xp[b] = (const bf16*) a.x + (size_t) r * a.ldx + (size_t) (a.segs ? 0 : group) * a.x_group_stride + 8 * t;
-    }
-    float acc[MT][NB][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int b = 0; b < NB; ++b)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) acc[m][b][i] = 0.0f;
-    for (int st0 = warp; st0 < steps; st0 += U * SK_WARPS) {
-        if (st0 != warp) load_w(st0);
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int st = st0 + u * SK_WARPS;
-            if (st >= steps) break;
-#pragma unroll
-            for (int b = 0; b < NB; ++b) {
-                uint4 xv = make_uint4(0, 0, 0, 0);
-                if (live[b]) xv = *reinterpret_cast<const uint4*>(xp[b] + (size_t) st * 32);
-#pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    skd::mma_bf16(acc[m][b], wr[u][m][0].x, wr[u][m][1].x, wr[u][m][0].y, wr[u][m][1].y, xv.x, xv.y);
-                    skd::mma_bf16(acc[m][b], wr[u][m][0].z, wr[u][m][1].z, wr[u][m][0].w, wr[u][m][1].w, xv.z, xv.w);
-                }
+    __syncthreads();
+    const int tiles = (a.w_rows + RG_TILE - 1) / RG_TILE, chunks = (a.ldw + R::KC - 1) / R::KC;
+    const bool producer = warp == RG_WARPS;
+    if (!producer || a.segs) skd::pdl_wait();        // weights do not depend on the predecessor: the ring fills before the wait
+    const int units = tiles * (a.segs ? *a.n_segs : a.groups);
+
+    if (producer) {
+        if (lane != 0) return;
+        int it = 0;
+        bool ok = true;
+        for (int u = blockIdx.x; u < units && ok; u += gridDim.x) {
+            const int row = (a.segs ? a.segs[u / tiles].group : u / tiles) * a.w_rows + (u % tiles) * RG_TILE;
+            for (int c = 0; c < chunks; ++c, ++it) {
+                const int s = it % R::STAGES;
+                if (it >= R::STAGES && !(ok = skd::mbar_wait_bounded(empty + s, ((it / R::STAGES) + 1) & 1, timeout_flag))) break;
+                uint8_t* st = smem + s * R::STAGE;
+                skd::mbar_expect_tx(full + s, R::STAGE);
+                skd::tma_load_3d(st, &map_w, 0, row, c * R::KB, full + s);
+                if (DUAL) skd::tma_load_3d(st + R::MAT, &map_w2, 0, row, c * R::KB, full + s);
             }
         }
+        for (int j = max(0, it - R::STAGES); j < it; ++j)               // no copy outlives the CTA
+            if (!skd::mbar_wait_bounded(full + j % R::STAGES, (j / R::STAGES) & 1, timeout_flag)) break;
+        return;
     }
+    bool ok = true;
+    int it = 0, buf = 0;
+    for (int u = blockIdx.x; u < units; u += gridDim.x, buf ^= 1) {
+        int col_group = u / tiles, row0 = 0, n_rows = a.rows;
+        if (a.segs) { const RowSegment sg = a.segs[u / tiles]; col_group = 0; row0 = sg.start; n_rows = sg.count; }
+        const bf16* xp[NB];
+        bool live[NB];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int b = 0; b < NB; ++b) {      // acc[0], [1]: output row g, activation rows 2t, 2t+1; acc[2], [3]: output row g + 8
-            float* p = part[warp][m][b];
-            p[(2 * t) * SK_TILE + g] = acc[m][b][0]; p[(2 * t + 1) * SK_TILE + g] = acc[m][b][1];
-            p[(2 * t) * SK_TILE + g + 8] = acc[m][b][2]; p[(2 * t + 1) * SK_TILE + g + 8] = acc[m][b][3];
+        for (int b = 0; b < NB; ++b) {
+            const int n = b * 8 + g;
+            live[b] = n < n_rows;
+            const int r = live[b] ? (a.row_index ? a.row_index[row0 + n] : row0 + n) : 0;
+            xp[b] = (const bf16*) a.x + (size_t) r * a.ldx + (size_t) col_group * a.x_group_stride;
         }
-    __syncthreads();
-    for (int i = threadIdx.x; i < NB * 8 * SK_TILE; i += SK_WARPS * 32) {
-        const int o = i % SK_TILE, n = i / SK_TILE;
-        if (n >= n_rows || tile + o >= a.w_rows) continue;
-        float v = 0.0f, v2 = 0.0f;
+        float acc[MT][NB][4];
 #pragma unroll
-        for (int w = 0; w < SK_WARPS; ++w) {
-            v += part[w][0][n >> 3][(n & 7) * SK_TILE + o];
-            if (DUAL) v2 += part[w][MT - 1][n >> 3][(n & 7) * SK_TILE + o];
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int b = 0; b < NB; ++b)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) acc[m][b][i] = 0.0f;
+        // A warp takes k32 steps warp, warp + 8, .. of a stage: half h of block j, of whose eight 16-byte chunks lane t takes 2t + h,
+        // so that the rows of a quarter-warp meet different banks. The activation's fragments are fetched a stage ahead.
+        constexpr int PER = 2 * R::KB / RG_WARPS;
+        const int h = warp & 1, kb0 = warp >> 1;
+        uint4 xv[PER][NB], xn[PER][NB];
+        auto load_x = [&](uint4 (&x)[PER][NB], int c) {
+#pragma unroll
+            for (int p = 0; p < PER; ++p) {
+                const int k = (c * R::KB + kb0 + p * (RG_WARPS / 2)) * 64 + (2 * t + h) * 8;
+#pragma unroll
+                for (int b = 0; b < NB; ++b) x[p][b] = live[b] && k < a.ldw ? *reinterpret_cast<const uint4*>(xp[b] + k) : make_uint4(0, 0, 0, 0);
+            }
+        };
+        load_x(xn, 0);
+        for (int c = 0; c < chunks; ++c, ++it) {
+            const int s = it % R::STAGES;
+#pragma unroll
+            for (int p = 0; p < PER; ++p)
+#pragma unroll
+                for (int b = 0; b < NB; ++b) xv[p][b] = xn[p][b];
+            if (c + 1 < chunks) load_x(xn, c + 1);
+            ok = ok && skd::mbar_wait_bounded(full + s, (it / R::STAGES) & 1, timeout_flag);
+            if (ok) {
+                const uint8_t* st = smem + s * R::STAGE + g * 128 + (((2 * t + h) ^ g) << 4);       // rows g and g + 8 share the XOR
+#pragma unroll
+                for (int p = 0; p < PER; ++p) {
+                    const uint8_t* bl = st + (kb0 + p * (RG_WARPS / 2)) * RG_TILE * 128;
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        const uint4 w0 = skd::lds128(bl + m * R::MAT), w1 = skd::lds128(bl + m * R::MAT + 8 * 128);
+#pragma unroll
+                        for (int b = 0; b < NB; ++b) {
+                            skd::mma_bf16(acc[m][b], w0.x, w1.x, w0.y, w1.y, xv[p][b].x, xv[p][b].y);
+                            skd::mma_bf16(acc[m][b], w0.z, w1.z, w0.w, w1.w, xv[p][b].z, xv[p][b].w);
+                        }
+                    }
+                }
+            }
+            __syncwarp();
+            if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(skd::smem_u32(empty + s)) : "memory");
         }
-        const int r = row0 + n;
-        if (a.scale) { const float f = a.scale[(size_t) r * a.scale_ld + (a.segs ? 0 : group)]; v *= f; v2 *= f; }
-        const size_t at = (size_t) r * a.ldy + (size_t) (a.segs ? 0 : group) * a.y_group_stride + tile + o;
-        if (OUT == LIN_OUT_F32) ((float*) a.y)[at] = v;
-        else if (OUT == LIN_OUT_ACT) ((bf16*) a.y)[at] = __float2bfloat16_rn(v);
-        else ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::silu(v) * v2);
+        float* pb = part + (size_t) buf * RG_WARPS * MT * NB * RG_TILE * 8;
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {      // acc[0], [1]: output row g, activation rows 2t, 2t+1; acc[2], [3]: output row g + 8
+                float* p = pb + ((warp * MT + m) * NB + b) * RG_TILE * 8;
+                p[(2 * t) * RG_TILE + g] = acc[m][b][0]; p[(2 * t + 1) * RG_TILE + g] = acc[m][b][1];
+                p[(2 * t) * RG_TILE + g + 8] = acc[m][b][2]; p[(2 * t + 1) * RG_TILE + g + 8] = acc[m][b][3];
+            }
+        asm volatile("bar.sync 1, %0;" ::"n"(RG_WARPS * 32) : "memory");
+        const int tile = (u % tiles) * RG_TILE;
+        for (int i = threadIdx.x; i < NB * 8 * RG_TILE; i += RG_WARPS * 32) {
+            const int o = i % RG_TILE, n = i / RG_TILE;
+            if (n >= n_rows || tile + o >= a.w_rows) continue;
+            float v = 0.0f, v2 = 0.0f;
+#pragma unroll
+            for (int w = 0; w < RG_WARPS; ++w) {
+                v += pb[((w * MT) * NB + (n >> 3)) * RG_TILE * 8 + (n & 7) * RG_TILE + o];
+                if (DUAL) v2 += pb[((w * MT + MT - 1) * NB + (n >> 3)) * RG_TILE * 8 + (n & 7) * RG_TILE + o];
+            }
+            const int r = row0 + n;
+            if (a.scale) { const float f = a.scale[(size_t) r * a.scale_ld + col_group]; v *= f; v2 *= f; }
+            const size_t at = (size_t) r * a.ldy + (size_t) col_group * a.y_group_stride + tile + o;
+            if (OUT == LIN_OUT_F32) ((float*) a.y)[at] = v;
+            else if (OUT == LIN_OUT_ACT) ((bf16*) a.y)[at] = __float2bfloat16_rn(v);
+            else ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::silu(v) * v2);
+        }
     }
 }
 
@@ -208,11 +257,23 @@ __global__ void to_act_kernel(const float* __restrict__ x, int cols, T* __restri
         skd::store_act(out + (size_t) blockIdx.x * ld + i, i < cols ? x[(size_t) blockIdx.x * cols + i] : 0.0f);
 }
 
-template <int NB, int OUT, int U>
-int32_t run_skinny(const LinearArgs& a, cudaStream_t s) {
-    const dim3 grid((a.w_rows + SK_TILE - 1) / SK_TILE, a.segs ? a.max_segs : a.groups);
-    SK_CUDA(launch_pdl(linear_skinny_kernel<NB, OUT, U>, grid, dim3(SK_WARPS * 32), 0, s, a));
+template <int NB, int OUT>
+int32_t run_ring(const LinearArgs& a, cudaStream_t s) {
+    constexpr int bytes = ring_smem<OUT == LIN_OUT_SWIGLU ? 2 : 1, NB>();
+    const int64_t units = (int64_t) ((a.w_rows + RG_TILE - 1) / RG_TILE) * (a.segs ? a.max_segs : a.groups);
+    constexpr int KB = Ring<OUT == LIN_OUT_SWIGLU ? 2 : 1>::KB;
+    CUtensorMap mw, mw2;
+    SK_TRY(tensor_map_k_blocks(&mw, a.w, (int64_t) a.groups * a.w_rows, a.ldw, RG_TILE, KB));
+    if (OUT == LIN_OUT_SWIGLU) SK_TRY(tensor_map_k_blocks(&mw2, a.w2, (int64_t) a.groups * a.w_rows, a.ldw, RG_TILE, KB)); else mw2 = mw;
+    SK_TRY(ensure_dynamic_smem((const void*) linear_ring_kernel<NB, OUT>, bytes));
+    const int64_t slots = (int64_t) sm_count() * (bytes <= 112 * 1024 ? 2 : 1);
+    SK_CUDA(launch_pdl(linear_ring_kernel<NB, OUT>, dim3((unsigned) std::min<int64_t>(units, slots)), dim3(RG_THREADS), bytes, s, mw, mw2, a, device_timeout_flag()));
     return SKAINET_CUDA_OK;
+}
+template <int NB>
+int32_t run_ring_out(const LinearArgs& a, cudaStream_t s) {
+    if (a.out == LIN_OUT_SWIGLU) return run_ring<NB, LIN_OUT_SWIGLU>(a, s);
+    return a.out == LIN_OUT_ACT ? run_ring<NB, LIN_OUT_ACT>(a, s) : run_ring<NB, LIN_OUT_F32>(a, s);
 }
 template <int OUT>
 int32_t run_f32(const LinearArgs& a, cudaStream_t s) {
@@ -233,14 +294,8 @@ int32_t launch_linear_bf16(const LinearArgs& a, cudaStream_t s) {
         return a.out == LIN_OUT_SWIGLU ? run_f32<LIN_OUT_SWIGLU>(a, s) : run_f32<LIN_OUT_F32>(a, s);
     }
     const int rows = a.segs ? a.seg_rows : a.rows;
-    if (rows <= 8) {
-        if (a.out == LIN_OUT_SWIGLU) return run_skinny<1, LIN_OUT_SWIGLU, 4>(a, s);
-        return a.out == LIN_OUT_ACT ? run_skinny<1, LIN_OUT_ACT, 8>(a, s) : run_skinny<1, LIN_OUT_F32, 8>(a, s);
-    }
-    if (rows <= SKINNY_MAX_ROWS) {
-        if (a.out == LIN_OUT_SWIGLU) return run_skinny<2, LIN_OUT_SWIGLU, 4>(a, s);
-        return a.out == LIN_OUT_ACT ? run_skinny<2, LIN_OUT_ACT, 8>(a, s) : run_skinny<2, LIN_OUT_F32, 8>(a, s);
-    }
+    if (rows <= 8) return run_ring_out<1>(a, s);
+    if (rows <= RING_MAX_ROWS) return run_ring_out<2>(a, s);
     return launch_gemm_bf16_tc(a, s);
 }
 

@@ -45,7 +45,7 @@ struct LinearArgs {
 int32_t launch_linear_bf16(const LinearArgs& a, cudaStream_t s);
 
 // Rows (plain and per-group) up to which the streaming kernel is used, and the segment length it takes.
-constexpr int SKINNY_MAX_ROWS = 16, SKINNY_SEG_ROWS = 8;
+constexpr int RING_MAX_ROWS = 16, RING_SEG_ROWS = 8;
 
 // gemm_bf16_tc.cu
 int32_t launch_gemm_bf16_tc(const LinearArgs& a, cudaStream_t s);

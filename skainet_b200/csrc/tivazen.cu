@@ -233,11 +233,11 @@ int32_t Tivazen::feed_forward(TvLayer& L, int rows, cudaStream_t s) {
         SK_TRY(launch_linear_bf16(l, s));
         // short runs stream their expert's weights past a few rows at a time, long ones go to the tensor-core tiles
         const int slots = rows * c.top, per = slots / c.experts;
-        const int seg_rows = f32 ? 32 : per <= 4 ? SKINNY_SEG_ROWS : per <= 24 ? 32 : 128;
+        const int seg_rows = f32 ? 32 : per <= 4 ? RING_SEG_ROWS : per <= 24 ? 32 : 128;
         SK_TRY(launch_route(z, rows, c.experts, c.top, seg_rows, route, s));
         l.segs = route.segs; l.n_segs = route.n_segs; l.seg_rows = seg_rows; l.max_segs = route_max_segs(slots, c.experts, seg_rows);
         l.groups = c.experts; l.rows = slots; l.scale = route.sorted_weight; l.scale_ld = 1;      // the weight multiplies the expert's input
-        if (f32 || seg_rows <= SKINNY_MAX_ROWS) l.row_index = route.sorted_row;
+        if (f32 || seg_rows <= RING_MAX_ROWS) l.row_index = route.sorted_row;
         else {
             SK_TRY(launch_gather_rows(act, route.sorted_row, act_sorted, slots, width_ld, f32, s));
             l.x = act_sorted; l.x_rows_alloc = max_slots;

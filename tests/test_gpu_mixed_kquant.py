@@ -54,8 +54,9 @@ def test_mixed_q4k_q6k_model_follows_the_cpu_composer(gpu, oracle, mixed_v):
         logits = cpu.step(tok)
         tin[0] = tok
         m.decode(tin, tout)
-    # the same bar as the teacher-forced test of the single-encoding models: drift stays at the level of single rounding flips
-    assert max(errs) < 0.15 and np.median(errs) < 0.02, errs
+    # exact to fp32 rounding until the first activation code that rounds the other way, which both variants reach only after the
+    # prompt; from there the drift stays at the level of single rounding flips, the bar of the single-encoding models
+    assert errs[0] < 1e-4 and max(errs) < 0.15, errs
     # batched rows (prefill chunk) and single rows agree: the part-wise projections scatter into the merged layout correctly
     m.reset()
     for t in prompt:
