@@ -190,11 +190,13 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 float u[32], v[32];
                 tmem_ld32(src + c0, u);
                 if (NA == 2) tmem_ld32(src + BN + c0, v);
+                // lane j fetches the factor of column j once; a load per column in the loop below would serialise on its latency
+                const float fl = a.scale && c0 + lane < tl.n_valid ? a.scale[(size_t) (tl.x_row + c0 + lane) * a.scale_ld + tl.col_group] : 1.0f;
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
+                    const float f = __shfl_sync(~0u, fl, j);
                     if (c0 + j >= tl.n_valid) break;
                     const int r = tl.x_row + c0 + j;
-                    const float f = a.scale ? a.scale[(size_t) r * a.scale_ld + tl.col_group] : 1.0f;
                     const size_t at = (size_t) r * a.ldy + (size_t) tl.col_group * a.y_group_stride + wr;
                     if (OUT == LIN_OUT_SWIGLU) {
                         if (wr < a.w_rows) ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::silu(u[j] * f) * (v[j] * f));
@@ -252,7 +254,7 @@ int32_t launch_gemm_bf16_tc(const LinearArgs& l, cudaStream_t s) {
     if (l.out == LIN_OUT_SWIGLU) return rows <= 32 ? run_tc<2, 32, LIN_OUT_SWIGLU>(l, s) : run_tc<2, 128, LIN_OUT_SWIGLU>(l, s);
     if (rows <= 32) return run_out<1, 32>(l, s);
     const int64_t wide = (int64_t) ((l.w_rows + 2 * BM - 1) / (2 * BM)) * (l.segs ? l.max_segs : (int64_t) ((l.rows + 127) / 128) * l.groups);
-    return l.w_rows > BM && wide >= sm_count() ? run_out<2, 128>(l, s) : run_out<1, 128>(l, s);
+    return l.w_rows > BM && wide * 5 >= (int64_t) sm_count() * 4 ? run_out<2, 128>(l, s) : run_out<1, 128>(l, s);
 }
 
 }  // namespace sk

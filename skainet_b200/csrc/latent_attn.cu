@@ -67,6 +67,9 @@ __device__ __forceinline__ void rotate_query(const LatentArgs& a, int row, int h
     skd::store_act(dst + i, o.x); skd::store_act(dst + i + half, o.y);
 }
 
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(skd::pack_bf16(v.x, v.y), skd::pack_bf16(v.z, v.w)); }
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a) {
     __shared__ float sh[8];
@@ -75,11 +78,19 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a) {
     const LatentGeom& g = a.g;
     const int row = blockIdx.x, half = g.rot_dim >> 1, hd = g.dim + g.rot_dim, pos = a.map.pos_of(row);
     const float* p = a.proj + (size_t) row * a.proj_ld;
-    for (int h = threadIdx.x >> 5; h < g.heads; h += 8) {
-        T* qn = (T*) a.qn + ((size_t) row * g.heads + h) * g.dim_ld();
-        for (int i = threadIdx.x & 31; i < g.dim; i += 32) skd::store_act(qn + i, p[(size_t) h * hd + i]);
-        for (int i = threadIdx.x & 31; i < half; i += 32) rotate_query<T>(a, row, h, i, pos);
-    }
+    if (g.dim % 4 == 0 && hd % 4 == 0 && a.proj_ld % 4 == 0) {         // rows 16-byte aligned: four elements per thread
+        const int q4 = g.dim >> 2;
+        for (int i = threadIdx.x; i < g.heads * q4; i += 256) {
+            const int h = i / q4, c = (i - h * q4) * 4;
+            const float4 v = *reinterpret_cast<const float4*>(p + (size_t) h * hd + c);
+            store4((T*) a.qn + ((size_t) row * g.heads + h) * g.dim_ld() + c, v);
+        }
+    } else
+        for (int i = threadIdx.x; i < g.heads * g.dim; i += 256) {
+            const int h = i / g.dim, c = i - h * g.dim;
+            skd::store_act((T*) a.qn + ((size_t) row * g.heads + h) * g.dim_ld() + c, p[(size_t) h * hd + c]);
+        }
+    for (int i = threadIdx.x; i < g.heads * half; i += 256) { const int h = i / half; rotate_query<T>(a, row, h, i - h * half, pos); }
     prep_row<T>(a, row, sh);
 }
 
@@ -196,7 +207,7 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
     float* red_l = red_m + NW * ROWS;
     int* qpos = (int*) (red_l + NW * ROWS);                   // position of each MMA row, -1: none
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mw = warp % MW, nw = warp / MW;
-    const int split = blockIdx.x, h0 = blockIdx.y * sp.heads_per_block, r0 = blockIdx.z * sp.rows_per_block;
+    const int split = blockIdx.x, h0 = blockIdx.y * sp.heads_per_block, r0 = (gridDim.z - 1 - blockIdx.z) * sp.rows_per_block;   // the rows with the most keys first
     const int hb = sp.heads_per_block;
     skd::pdl_launch_dependents();
     skd::pdl_wait();
@@ -253,12 +264,27 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
         // KT = 2: one ldmatrix covers both key tiles of a k16 step; KT = 1: two k16 steps of the one key tile
         if (KT == 2) {
             const bf16* bk = kt + (nw * 16 + (lane & 7) + ((lane >> 4) << 3)) * sld + ((lane >> 3) & 1) * 8;
-            for (int k = 0; k < kld; k += 16) {
+            float s2[KT][4] = {};                             // second pair of accumulators: four independent chains
+            int k = 0;
+            for (; k + 64 <= kld; k += 64) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    uint32_t fa[4], fb[4];
+                    ldsm4(fa, aq + k + 16 * j); ldsm4(fb, bk + k + 16 * j);
+                    skd::mma_bf16(j & 1 ? s2[0] : s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
+                    skd::mma_bf16(j & 1 ? s2[KT - 1] : s4[KT - 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
+                }
+            }
+            for (; k < kld; k += 16) {
                 uint32_t fa[4], fb[4];
                 ldsm4(fa, aq + k); ldsm4(fb, bk + k);
                 skd::mma_bf16(s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
                 skd::mma_bf16(s4[KT - 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
             }
+#pragma unroll
+            for (int i = 0; i < KT; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) s4[i][j] += s2[i][j];
         } else {
             const bf16* bk = kt + (nw * 8 + (lane & 7)) * sld + (lane >> 3) * 8;
             float s1[4] = {}, s2[4] = {}, s3[4] = {};         // four independent accumulator chains
