@@ -182,10 +182,12 @@ __device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(skd::smem_u32(p)) : "memory");
 }
 
-// MW warps over 16-row groups x NW = 8 / MW warps over keys (scores) and over 16-column groups of the latent (mix, NT each).
+// MW warps over 16-row groups x NW warps over keys (scores, eight each) and over 16-column groups of the latent (mix, NT each).
+// The scores and the mix are chains of dependent shared-memory loads and MMAs: with 64 rows, sixteen warps hide them better than
+// eight that own twice the columns (304 -> 279 us for 1024 rows x 32 heads at a latent of 512).
 template <int MW>
 struct AttnShape {
-    static constexpr int NW = 8 / MW, KT = MW == 4 ? 2 : 1, BK = NW * KT * 8, ROWS = 16 * MW;
+    static constexpr int WARPS = MW == 4 ? 16 : 8, THREADS = WARPS * 32, NW = WARPS / MW, BK = NW * 8, ROWS = 16 * MW;
     static int smem(int key_ld, int stages) {
         return (ROWS + stages * BK) * (key_ld + 8) * 2 + ROWS * (BK + 8) * 2 + (2 * NW * ROWS + ROWS) * 4;
     }
@@ -193,10 +195,10 @@ struct AttnShape {
 constexpr int ATTN_MAX_SMEM = 225 * 1024;
 
 template <int MW, int NT, int ST>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(AttnShape<MW>::THREADS)
 latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
     typedef AttnShape<MW> S;
-    constexpr int NW = S::NW, KT = S::KT, BK = S::BK, ROWS = S::ROWS;
+    constexpr int NW = S::NW, BK = S::BK, ROWS = S::ROWS;
     extern __shared__ __align__(16) uint8_t smem[];
     const LatentGeom& g = a.g;
     const int kld = g.key_ld(), sld = kld + 8, RP = g.rank_pad(), chunks = kld >> 3;
@@ -221,7 +223,7 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
     auto fetch = [&](int t) {                                 // keys past hi repeat the newest one; their weights are masked
         if (t < t1) {
             bf16* dst = sk_ + (t % ST) * BK * sld;
-            for (int j = warp; j < BK; j += 8) {
+            for (int j = warp; j < BK; j += S::WARPS) {
                 const int p = min(lo + t * BK + j, hi);
                 const bf16* src = cache + (size_t) (p % a.cache.cap) * kld;
                 for (int c = lane; c < chunks; c += 32) cp16(dst + j * sld + c * 8, src + c * 8);
@@ -230,7 +232,7 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     for (int i = 0; i < ST - 1; ++i) fetch(t0 + i);
-    for (int m = warp; m < ROWS; m += 8) {                    // query rows, zero where there is none
+    for (int m = warp; m < ROWS; m += S::WARPS) {             // query rows, zero where there is none
         const int r = r0 + m / hb, h = h0 + m % hb;
         const bool live = m < sp.rows_per_block * hb && r <= r_last && h < g.heads;
         if (lane == 0) qpos[m] = live ? a.map.pos_of(r) : -1;
@@ -256,43 +258,14 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
         __syncthreads();                                      // tile t is staged; every warp is done with tile t - 1
         fetch(t + ST - 1);
         const bf16* kt = sk_ + (t % ST) * BK * sld;
-        float s4[KT][4];
-#pragma unroll
-        for (int i = 0; i < KT; ++i)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) s4[i][j] = 0.0f;
-        // KT = 2: one ldmatrix covers both key tiles of a k16 step; KT = 1: two k16 steps of the one key tile
-        if (KT == 2) {
-            const bf16* bk = kt + (nw * 16 + (lane & 7) + ((lane >> 4) << 3)) * sld + ((lane >> 3) & 1) * 8;
-            float s2[KT][4] = {};                             // second pair of accumulators: four independent chains
-            int k = 0;
-            for (; k + 64 <= kld; k += 64) {
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    uint32_t fa[4], fb[4];
-                    ldsm4(fa, aq + k + 16 * j); ldsm4(fb, bk + k + 16 * j);
-                    skd::mma_bf16(j & 1 ? s2[0] : s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
-                    skd::mma_bf16(j & 1 ? s2[KT - 1] : s4[KT - 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
-                }
-            }
-            for (; k < kld; k += 16) {
-                uint32_t fa[4], fb[4];
-                ldsm4(fa, aq + k); ldsm4(fb, bk + k);
-                skd::mma_bf16(s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
-                skd::mma_bf16(s4[KT - 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
-            }
-#pragma unroll
-            for (int i = 0; i < KT; ++i)
-#pragma unroll
-                for (int j = 0; j < 4; ++j) s4[i][j] += s2[i][j];
-        } else {
+        float s4[4] = {}, s1[4] = {}, s2[4] = {}, s3[4] = {};         // four independent accumulator chains
+        {
             const bf16* bk = kt + (nw * 8 + (lane & 7)) * sld + (lane >> 3) * 8;
-            float s1[4] = {}, s2[4] = {}, s3[4] = {};         // four independent accumulator chains
             int k = 0;
             for (; k + 64 <= kld; k += 64) {
                 uint32_t fa[4], fb[4];
                 ldsm4(fb, bk + k); ldsm4(fa, aq + k);
-                skd::mma_bf16(s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
+                skd::mma_bf16(s4, fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
                 ldsm4(fa, aq + k + 16);
                 skd::mma_bf16(s1, fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
                 ldsm4(fb, bk + k + 32); ldsm4(fa, aq + k + 32);
@@ -305,23 +278,21 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
                 ldsm4(fa, aq + k);
                 asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(fb[0]), "=r"(fb[1])
                              : "r"(skd::smem_u32(kt + (nw * 8 + (lane & 7)) * sld + ((lane >> 3) & 1) * 8 + k)) : "memory");
-                skd::mma_bf16(s4[0], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
+                skd::mma_bf16(s4, fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
             }
 #pragma unroll
-            for (int j = 0; j < 4; ++j) s4[0][j] += s1[j] + (s2[j] + s3[j]);
+            for (int j = 0; j < 4; ++j) s4[j] += s1[j] + (s2[j] + s3[j]);
         }
         // scaled scores in powers of two, masked; row maxima over this warp's keys, then over the warps
         const int pa = qpos[ra], pb = qpos[rb];
         float mx[2] = {NEG_BIG, NEG_BIG};
 #pragma unroll
-        for (int i = 0; i < KT; ++i)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int key = lo + t * BK + (nw * KT + i) * 8 + 2 * (lane & 3) + (j & 1), p = j < 2 ? pa : pb;
-                const float v = key <= p && p - key < a.window ? s4[i][j] * sc : -INFINITY;
-                s4[i][j] = v;
-                mx[j >> 1] = fmaxf(mx[j >> 1], v);
-            }
+        for (int j = 0; j < 4; ++j) {
+            const int key = lo + t * BK + nw * 8 + 2 * (lane & 3) + (j & 1), p = j < 2 ? pa : pb;
+            const float v = key <= p && p - key < a.window ? s4[j] * sc : -INFINITY;
+            s4[j] = v;
+            mx[j >> 1] = fmaxf(mx[j >> 1], v);
+        }
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             mx[r] = fmaxf(mx[r], __shfl_xor_sync(~0u, mx[r], 1)); mx[r] = fmaxf(mx[r], __shfl_xor_sync(~0u, mx[r], 2));
@@ -337,15 +308,15 @@ latent_attn_mma_kernel(const LatentArgs a, const SplitArgs sp) {
             al[r] = exp2f(m_run[r] - m);
             m_run[r] = m; l_run[r] *= al[r];
         }
-#pragma unroll
-        for (int i = 0; i < KT; ++i) {
-            const float e0 = exp2f(s4[i][0] - m_run[0]), e1 = exp2f(s4[i][1] - m_run[0]), e2 = exp2f(s4[i][2] - m_run[1]), e3 = exp2f(s4[i][3] - m_run[1]);
+        {
+            const float e0 = exp2f(s4[0] - m_run[0]), e1 = exp2f(s4[1] - m_run[0]), e2 = exp2f(s4[2] - m_run[1]), e3 = exp2f(s4[3] - m_run[1]);
             l_run[0] += e0 + e1; l_run[1] += e2 + e3;
-            const int c = (nw * KT + i) * 8 + 2 * (lane & 3);
+            const int c = nw * 8 + 2 * (lane & 3);
             *(uint32_t*) (spb + ra * (BK + 8) + c) = skd::pack_bf16(e0, e1);
             *(uint32_t*) (spb + rb * (BK + 8) + c) = skd::pack_bf16(e2, e3);
         }
         __syncthreads();
+        if (__any_sync(~0u, al[0] != 1.0f || al[1] != 1.0f))             // a running maximum moved
 #pragma unroll
         for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -538,30 +509,29 @@ __global__ void transpose_heads_kernel(const bf16* __restrict__ src, bf16* __res
     }
 }
 
-template <int MW, int NT>
-int32_t run_mma(const LatentArgs& a, const SplitArgs& sp, dim3 grid, cudaStream_t s) {
-    typedef AttnShape<MW> S;
-    if (S::smem(a.g.key_ld(), 3) <= ATTN_MAX_SMEM) {
-        const int bytes = S::smem(a.g.key_ld(), 3);
-        SK_TRY(ensure_dynamic_smem((const void*) latent_attn_mma_kernel<MW, NT, 3>, bytes));
-        SK_CUDA(launch_pdl(latent_attn_mma_kernel<MW, NT, 3>, grid, dim3(256), bytes, s, a, sp));
-        return SKAINET_CUDA_OK;
-    }
-    const int bytes = S::smem(a.g.key_ld(), 2);
-    SK_TRY(ensure_dynamic_smem((const void*) latent_attn_mma_kernel<MW, NT, 2>, bytes));
-    SK_CUDA(launch_pdl(latent_attn_mma_kernel<MW, NT, 2>, grid, dim3(256), bytes, s, a, sp));
+template <int MW, int NT, int ST>
+int32_t run_mma_st(const LatentArgs& a, const SplitArgs& sp, dim3 grid, cudaStream_t s) {
+    const int bytes = AttnShape<MW>::smem(a.g.key_ld(), ST);
+    SK_TRY(ensure_dynamic_smem((const void*) latent_attn_mma_kernel<MW, NT, ST>, bytes));
+    SK_CUDA(launch_pdl(latent_attn_mma_kernel<MW, NT, ST>, grid, dim3(AttnShape<MW>::THREADS), bytes, s, a, sp));
     return SKAINET_CUDA_OK;
 }
-
-bool mma_fits(const LatentGeom& g, int mw) {
-    const int nw = 8 / mw, nt = (g.rank_pad() / 16 + nw - 1) / nw;
-    return nt <= (mw == 4 ? 16 : 8) && (mw == 4 ? AttnShape<4>::smem(g.key_ld(), 2) : AttnShape<1>::smem(g.key_ld(), 2)) <= ATTN_MAX_SMEM;
+template <int MW, int NT>
+int32_t run_mma(const LatentArgs& a, const SplitArgs& sp, dim3 grid, cudaStream_t s) {
+    return AttnShape<MW>::smem(a.g.key_ld(), 3) <= ATTN_MAX_SMEM ? run_mma_st<MW, NT, 3>(a, sp, grid, s) : run_mma_st<MW, NT, 2>(a, sp, grid, s);
 }
 
-int32_t launch_mma(const LatentArgs& a, const SplitArgs& sp, int mw, dim3 grid, cudaStream_t s) {
-    const int nw = 8 / mw, nt = (a.g.rank_pad() / 16 + nw - 1) / nw;
-    if (mw == 1) return nt <= 1 ? run_mma<1, 1>(a, sp, grid, s) : nt <= 2 ? run_mma<1, 2>(a, sp, grid, s) : nt <= 4 ? run_mma<1, 4>(a, sp, grid, s) : run_mma<1, 8>(a, sp, grid, s);
-    return nt <= 2 ? run_mma<4, 2>(a, sp, grid, s) : nt <= 4 ? run_mma<4, 4>(a, sp, grid, s) : nt <= 8 ? run_mma<4, 8>(a, sp, grid, s) : run_mma<4, 16>(a, sp, grid, s);
+// 16-column groups of the latent per warp; 0: the tile kernel does not take this geometry.
+template <int MW>
+int mma_groups(const LatentGeom& g) {
+    typedef AttnShape<MW> S;
+    const int nt = (g.rank_pad() / 16 + S::NW - 1) / S::NW;
+    return nt <= 8 && S::smem(g.key_ld(), 2) <= ATTN_MAX_SMEM ? nt : 0;
+}
+template <int MW>
+int32_t launch_mma(const LatentArgs& a, const SplitArgs& sp, dim3 grid, cudaStream_t s) {
+    const int nt = mma_groups<MW>(a.g);
+    return nt <= 1 ? run_mma<MW, 1>(a, sp, grid, s) : nt <= 2 ? run_mma<MW, 2>(a, sp, grid, s) : nt <= 4 ? run_mma<MW, 4>(a, sp, grid, s) : run_mma<MW, 8>(a, sp, grid, s);
 }
 
 }  // namespace
@@ -585,7 +555,7 @@ int32_t launch_latent_attention(const LatentArgs& args, cudaStream_t s) {
     // key splits: enough CTAs for the machine, no more than there are key tiles, records within the scratch
     const bool small = a.map.seq < 0 || a.rows <= LATENT_FUSED_ROWS;      // rows of different sequences share no keys
     const int mw = small ? 1 : 4;
-    const bool mma = !a.f32_act && mma_fits(g, mw);
+    const bool mma = !a.f32_act && (mw == 4 ? mma_groups<4>(g) : mma_groups<1>(g)) > 0;
     SplitArgs sp = {1, 1, 1};
     dim3 grid;
     int bk = ROWS_BK;
@@ -601,7 +571,7 @@ int32_t launch_latent_attention(const LatentArgs& args, cudaStream_t s) {
     sp.n_splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) sm_count() / std::max<int64_t>(1, blocks), (int64_t) (tiles + 1) / 2, MERGE_MAX_SPLITS, LATENT_PART_RECORDS / std::max<int64_t>(1, records)}));
     grid.x = sp.n_splits;
     if (!few && sp.n_splits == 1) a.part = nullptr;
-    if (mma) SK_TRY(launch_mma(a, sp, mw, grid, s));
+    if (mma) SK_TRY(mw == 4 ? launch_mma<4>(a, sp, grid, s) : launch_mma<1>(a, sp, grid, s));
     else {
         const int bytes = (g.key_ld() + g.rank_pad()) * (int) sizeof(float);
         if (a.f32_act) {
