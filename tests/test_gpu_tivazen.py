@@ -25,6 +25,8 @@ CONFIGS = {
     "heads": M.config([(A(heads=20, dim=32, rot_dim=16, vdim=24, kv_rank=64, window=70), D(96)), (A(heads=70, dim=8, rot_dim=4, vdim=6, kv_rank=40, window=150), X(16, 1, 40))], width=128, vocab=300),
     # the widest latent the tile kernel holds, and one beyond it
     "wide": M.config([(A(heads=4, dim=64, rot_dim=64, vdim=40, kv_rank=512, window=33, scale=0.05), D(64)), (A(heads=3, dim=16, rot_dim=8, vdim=20, kv_rank=560, window=50, scale=0.05), None)], width=96, vocab=130),
+    # nothing a multiple of anything: scalar paths of the row kernels, ragged tiles everywhere
+    "odd": M.config([(A(heads=3, dim=7, rot_dim=2, vdim=5, kv_rank=17, window=11), D(35)), (A(heads=7, dim=5, rot_dim=2, vdim=3, kv_rank=17, window=29, kv_from=0), X(9, 4, 13)), (A(heads=2, dim=1, rot_dim=4, vdim=9, kv_rank=13, window=300), None)], width=67, vocab=101),
     "plain": M.config([(A(heads=8, dim=16, rot_dim=8, vdim=16, kv_rank=48, window=40), D(64)), (A(heads=8, dim=16, rot_dim=8, vdim=16, kv_rank=48, window=40), X(8, 2, 32))], width=64, vocab=150),
 }
 
