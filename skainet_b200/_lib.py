@@ -123,6 +123,11 @@ SIGNATURES = {
     "skainet_cuda_tivazen_set_weight": [i64, i32, i32, i32, i64],
     "skainet_cuda_tivazen_set_vector": [i64, i32, i32, f32p, i32],
     "skainet_cuda_tivazen_synth": [i64, C.c_uint64, f32],
+    # include/skainet_cuda_fomalix.h
+    "skainet_cuda_fomalix_create": [vp, vp, i64p],
+    "skainet_cuda_fomalix_set_weight": [i64, i32, i32, i64],
+    "skainet_cuda_fomalix_set_vector": [i64, i32, i32, f32p, i32],
+    "skainet_cuda_fomalix_synth": [i64, C.c_uint64, f32],
 }
 _RESTYPE = {"skainet_cuda_last_error": C.c_char_p, "skainet_cuda_version": C.c_char_p}
 

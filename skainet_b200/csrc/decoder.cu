@@ -1,6 +1,6 @@
 // The decoder runtime shared by every model design (contract: decoder.cuh, include/skainet_cuda_llama.h): the step graph with
 // greedy sampling, chunked prompts, logits of chosen positions, generation on the device. What a layer computes is the
-// design's (llama.cu, tivazen.cu).
+// design's (llama.cu, tivazen.cu, fomalix.cu).
 #include "decoder.cuh"
 #include "tma.cuh"
 
@@ -181,7 +181,15 @@ int32_t decoder_init(Decoder* m) {
     return SKAINET_CUDA_OK;
 }
 
+int32_t Decoder::alloc(void** p, size_t bytes) {
+    SK_CUDA(cudaMalloc(p, std::max<size_t>(bytes, 16)));
+    owned.push_back(*p);
+    SK_CUDA(cudaMemset(*p, 0, std::max<size_t>(bytes, 16)));
+    return SKAINET_CUDA_OK;
+}
+
 Decoder::~Decoder() {
+    for (void* p : owned) cudaFree(p);
     for (auto& kv : graphs) cudaGraphExecDestroy(kv.second);
     for (void* p : {(void*) logits, (void*) logits_full, (void*) pairs, (void*) cur_token, (void*) pos, (void*) kv_len, (void*) log, (void*) log_cursor})
         if (p) cudaFree(p);

@@ -34,6 +34,11 @@ struct Decoder {
     int* d_flag = nullptr;         // the device's bounded-wait flag (owned by the library, not by the model)
     int* h_flag = nullptr;         // pinned host copy read after every synchronising call
     uint64_t magic = 0;
+    std::vector<void*> owned;      // device allocations freed with the model
+
+    // Zeroed: the tails of activation rows and cache rows are read as zeros and never written.
+    int32_t alloc(void** p, size_t bytes);
+    template <typename T> int32_t alloc(T** p, size_t count) { return alloc((void**) p, count * sizeof(T)); }
 
     virtual ~Decoder();
     virtual int32_t finalize() = 0;

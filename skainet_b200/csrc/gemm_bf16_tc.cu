@@ -9,7 +9,7 @@
 //   warp 1     one lane issues the MMAs and commits (stage barriers to the producer, accumulator barrier to the epilogue)
 //   warps 2-5  epilogue: TMEM -> registers -> global; two accumulator sets, so it overlaps the next tile's MMAs
 // NA = 2 keeps two 128-row weight tiles per activation tile: twice the rows of one matrix, or the same rows of gate and up,
-// whose product silu(gate) * up is then formed in the epilogue without a round trip.
+// whose product act(gate) * up is then formed in the epilogue without a round trip.
 // Every mbarrier wait is bounded; a wait that runs out raises the device flag and the CTA still frees its TMEM.
 #include "linear_bf16.cuh"
 #include "tensor_map.cuh"
@@ -198,8 +198,8 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     if (c0 + j >= tl.n_valid) break;
                     const int r = tl.x_row + c0 + j;
                     const size_t at = (size_t) r * a.ldy + (size_t) tl.col_group * a.y_group_stride + wr;
-                    if (OUT == LIN_OUT_SWIGLU) {
-                        if (wr < a.w_rows) ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::silu(u[j] * f) * (v[j] * f));
+                    if (lin_gated(OUT)) {
+                        if (wr < a.w_rows) ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::lin_gate<OUT>(u[j] * f) * (v[j] * f));
                     } else {
                         if (wr < a.w_rows) { if (OUT == LIN_OUT_F32) ((float*) a.y)[at] = u[j] * f; else ((bf16*) a.y)[at] = __float2bfloat16_rn(u[j] * f); }
                         if (NA == 2 && wr + BM < a.w_rows) { if (OUT == LIN_OUT_F32) ((float*) a.y)[at + BM] = v[j] * f; else ((bf16*) a.y)[at + BM] = __float2bfloat16_rn(v[j] * f); }
@@ -222,13 +222,13 @@ int32_t run_tc(const LinearArgs& l, cudaStream_t s) {
     CUtensorMap ma, ma2, mb;
     const int64_t w_total = (int64_t) l.groups * l.w_rows;
     SK_TRY(tensor_map_rows(&ma, l.w, w_total, l.ldw, BM));
-    if (OUT == LIN_OUT_SWIGLU) SK_TRY(tensor_map_rows(&ma2, l.w2, w_total, l.ldw, BM)); else ma2 = ma;
+    if (lin_gated(OUT)) SK_TRY(tensor_map_rows(&ma2, l.w2, w_total, l.ldw, BM)); else ma2 = ma;
     SK_TRY(tensor_map_rows(&mb, (const bf16*) l.x, l.x_rows_alloc, l.ldx, BN));
     TcArgs a = {};
     a.y = l.y; a.ldy = l.ldy; a.y_group_stride = l.y_group_stride; a.scale = l.scale; a.scale_ld = l.scale_ld;
     a.segs = l.segs; a.n_segs = l.n_segs; a.w_rows = l.w_rows; a.rows = l.rows; a.groups = l.groups;
     a.ksteps = l.ldw / BKE; a.x_group_stride = l.x_group_stride;
-    a.a2_rows = (NA == 2 && OUT != LIN_OUT_SWIGLU) ? BM : 0;
+    a.a2_rows = (NA == 2 && !lin_gated(OUT)) ? BM : 0;
     a.m_tiles = (l.w_rows + BM + a.a2_rows - 1) / (BM + a.a2_rows);
     a.n_tiles = (l.rows + BN - 1) / BN;
     a.timeout_flag = device_timeout_flag();
@@ -251,6 +251,7 @@ int32_t launch_gemm_bf16_tc(const LinearArgs& l, cudaStream_t s) {
     SK_REQUIRE(!l.f32_act && l.row_index == nullptr, "gemm_bf16_tc: bf16 rows in order only");
     const int rows = l.segs ? l.seg_rows : l.rows;
     // a segment's rows past its end belong to the next one: their columns are computed and not stored
+    if (l.out == LIN_OUT_GEGLU) return rows <= 32 ? run_tc<2, 32, LIN_OUT_GEGLU>(l, s) : run_tc<2, 128, LIN_OUT_GEGLU>(l, s);
     if (l.out == LIN_OUT_SWIGLU) return rows <= 32 ? run_tc<2, 32, LIN_OUT_SWIGLU>(l, s) : run_tc<2, 128, LIN_OUT_SWIGLU>(l, s);
     if (rows <= 32) return run_out<1, 32>(l, s);
     const int64_t wide = (int64_t) ((l.w_rows + 2 * BM - 1) / (2 * BM)) * (l.segs ? l.max_segs : (int64_t) ((l.rows + 127) / 128) * l.groups);

@@ -8,6 +8,7 @@
 // one [latent | rotated part] row per key for all heads, and a cached row is never expanded.
 #pragma once
 #include "linear_bf16.cuh"
+#include "rowmap.cuh"
 
 namespace sk {
 
@@ -25,16 +26,6 @@ struct LatentGeom {                       // what the buffers of a layer are lai
         for (int i = 0; i < 5; ++i) if (a[i] != b[i]) return a[i] < b[i];
         return false;
     }
-};
-
-// Which sequence and position an activation row stands for: seq >= 0, consecutive tokens of that sequence from pos[seq];
-// seq < 0, row b is the next token of sequence b.
-struct RowMap {
-    const int32_t* pos; int seq;
-#ifdef __CUDACC__
-    __device__ __forceinline__ int seq_of(int row) const { return seq < 0 ? row : seq; }
-    __device__ __forceinline__ int pos_of(int row) const { return seq < 0 ? pos[row] : pos[seq] + row; }
-#endif
 };
 
 struct LatentCache {                      // one layer's rows; a ring of `cap` positions per sequence

@@ -36,7 +36,7 @@ constexpr int ring_smem() { return Ring<MT>::STAGES * Ring<MT>::STAGE + 2 * RG_W
 template <int NB, int OUT>
 __global__ void __launch_bounds__(RG_THREADS, 2)
 linear_ring_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_w2, const LinearArgs a, int* __restrict__ timeout_flag) {
-    constexpr bool DUAL = OUT == LIN_OUT_SWIGLU;
+    constexpr bool DUAL = lin_gated(OUT);
     constexpr int MT = DUAL ? 2 : 1;
     typedef Ring<MT> R;
     extern __shared__ uint8_t raw[];
@@ -162,7 +162,7 @@ linear_ring_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             const size_t at = (size_t) r * a.ldy + (size_t) col_group * a.y_group_stride + tile + o;
             if (OUT == LIN_OUT_F32) ((float*) a.y)[at] = v;
             else if (OUT == LIN_OUT_ACT) ((bf16*) a.y)[at] = __float2bfloat16_rn(v);
-            else ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::silu(v) * v2);
+            else ((bf16*) a.y)[at] = __float2bfloat16_rn(skd::lin_gate<OUT>(v) * v2);
         }
     }
 }
@@ -172,7 +172,7 @@ constexpr int F_O = 64, F_N = 32, F_K = 32;
 template <int OUT>
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const LinearArgs a) {
-    constexpr bool DUAL = OUT == LIN_OUT_SWIGLU;
+    constexpr bool DUAL = lin_gated(OUT);
     __shared__ float sx[F_N][F_K + 1], sw[DUAL ? 2 : 1][F_O][F_K + 1];
     skd::pdl_launch_dependents();
     skd::pdl_wait();
@@ -234,7 +234,7 @@ linear_f32_kernel(const LinearArgs a) {
             const int o = o0 + to + 16 * i;
             if (o >= a.w_rows) continue;
             const float v = acc[0][i][j] * f;
-            ((float*) a.y)[(size_t) r * a.ldy + (size_t) col_group * a.y_group_stride + o] = DUAL ? skd::silu(v) * (acc[1][i][j] * f) : v;
+            ((float*) a.y)[(size_t) r * a.ldy + (size_t) col_group * a.y_group_stride + o] = DUAL ? skd::lin_gate<OUT>(v) * (acc[1][i][j] * f) : v;
         }
     }
 }
@@ -259,12 +259,12 @@ __global__ void to_act_kernel(const float* __restrict__ x, int cols, T* __restri
 
 template <int NB, int OUT>
 int32_t run_ring(const LinearArgs& a, cudaStream_t s) {
-    constexpr int bytes = ring_smem<OUT == LIN_OUT_SWIGLU ? 2 : 1, NB>();
+    constexpr int bytes = ring_smem<lin_gated(OUT) ? 2 : 1, NB>();
     const int64_t units = (int64_t) ((a.w_rows + RG_TILE - 1) / RG_TILE) * (a.segs ? a.max_segs : a.groups);
-    constexpr int KB = Ring<OUT == LIN_OUT_SWIGLU ? 2 : 1>::KB;
+    constexpr int KB = Ring<lin_gated(OUT) ? 2 : 1>::KB;
     CUtensorMap mw, mw2;
     SK_TRY(tensor_map_k_blocks(&mw, a.w, (int64_t) a.groups * a.w_rows, a.ldw, RG_TILE, KB));
-    if (OUT == LIN_OUT_SWIGLU) SK_TRY(tensor_map_k_blocks(&mw2, a.w2, (int64_t) a.groups * a.w_rows, a.ldw, RG_TILE, KB)); else mw2 = mw;
+    if (lin_gated(OUT)) SK_TRY(tensor_map_k_blocks(&mw2, a.w2, (int64_t) a.groups * a.w_rows, a.ldw, RG_TILE, KB)); else mw2 = mw;
     SK_TRY(ensure_dynamic_smem((const void*) linear_ring_kernel<NB, OUT>, bytes));
     const int64_t slots = (int64_t) sm_count() * (bytes <= 112 * 1024 ? 2 : 1);
     SK_CUDA(launch_pdl(linear_ring_kernel<NB, OUT>, dim3((unsigned) std::min<int64_t>(units, slots)), dim3(RG_THREADS), bytes, s, mw, mw2, a, device_timeout_flag()));
@@ -273,6 +273,7 @@ int32_t run_ring(const LinearArgs& a, cudaStream_t s) {
 template <int NB>
 int32_t run_ring_out(const LinearArgs& a, cudaStream_t s) {
     if (a.out == LIN_OUT_SWIGLU) return run_ring<NB, LIN_OUT_SWIGLU>(a, s);
+    if (a.out == LIN_OUT_GEGLU) return run_ring<NB, LIN_OUT_GEGLU>(a, s);
     return a.out == LIN_OUT_ACT ? run_ring<NB, LIN_OUT_ACT>(a, s) : run_ring<NB, LIN_OUT_F32>(a, s);
 }
 template <int OUT>
@@ -291,6 +292,7 @@ int32_t launch_linear_bf16(const LinearArgs& a, cudaStream_t s) {
     SK_REQUIRE((a.segs ? a.max_segs : a.groups) <= 65535, "linear_bf16: more than 65535 groups or segments");
     if (a.f32_act) {
         SK_REQUIRE((a.segs ? a.seg_rows : a.rows) <= 65535 * F_N, "linear_bf16: too many rows");
+        if (a.out == LIN_OUT_GEGLU) return run_f32<LIN_OUT_GEGLU>(a, s);
         return a.out == LIN_OUT_SWIGLU ? run_f32<LIN_OUT_SWIGLU>(a, s) : run_f32<LIN_OUT_F32>(a, s);
     }
     const int rows = a.segs ? a.seg_rows : a.rows;

@@ -18,10 +18,12 @@ constexpr int bf16_ld(int cols) { return (cols + 63) / 64 * 64; }
 // A run of activation rows that share one weight matrix: rows [start, start + count) take matrix `group`.
 struct RowSegment { int32_t group, start, count, pad; };
 
-enum { LIN_OUT_F32 = 0, LIN_OUT_ACT = 1, LIN_OUT_SWIGLU = 2 };   // fp32 rows | activation type | silu(W x) * (W2 x) in the activation type
+// fp32 rows | activation type | silu(W x) * (W2 x) | gelu(W x) * (W2 x), tanh form; the last two in the activation type
+enum { LIN_OUT_F32 = 0, LIN_OUT_ACT = 1, LIN_OUT_SWIGLU = 2, LIN_OUT_GEGLU = 3 };
+constexpr bool lin_gated(int out) { return out == LIN_OUT_SWIGLU || out == LIN_OUT_GEGLU; }
 
 struct LinearArgs {
-    const bf16 *w = nullptr, *w2 = nullptr;      // w2: the up matrix of LIN_OUT_SWIGLU
+    const bf16 *w = nullptr, *w2 = nullptr;      // w2: the up matrix of the gated outputs
     int w_rows = 0;                              // output rows of one group
     int ldw = 0;                                 // padded K
     int groups = 1;                              // matrices stacked in w, [groups][w_rows][ldw]
@@ -60,6 +62,9 @@ int32_t launch_to_act(const float* x, int rows, int cols, void* out, int ld, boo
 namespace skd {
 
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+// 0.5 z (1 + tanh(u)) = z / (1 + exp(-2u)), u = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) { return z / (1.0f + expf(-1.5957691216057308f * z * (1.0f + 0.044715f * z * z))); }
+template <int OUT> __device__ __forceinline__ float lin_gate(float v) { return OUT == sk::LIN_OUT_GEGLU ? gelu_tanh(v) : silu(v); }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ void store_act(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 __device__ __forceinline__ void store_act(float* p, float v) { *p = v; }

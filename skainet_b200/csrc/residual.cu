@@ -1,4 +1,4 @@
-// Residual, one-number norm and depth average (contract: residual.cuh). All HBM- or latency-bound: one pass over the row for
+// Residual, norms and depth average (contract: residual.cuh). All HBM- or latency-bound: one pass over the row for
 // the sum of squares, one that writes. With few rows a cluster of up to eight CTAs shares a row (the sum of squares through
 // distributed shared memory), because a late layer's average reads every earlier state of the row.
 #include "residual.cuh"
@@ -102,6 +102,112 @@ __global__ void __launch_bounds__(RT) sublayer_kernel(const SublayerArgs a) {
     if (cs > 1) cl.sync();                                      // no CTA leaves while its partial sum may still be read
 }
 
+// Sum of v over the CTA, then over the cluster's CTAs through distributed shared memory. `part` is written once per call site.
+__device__ __forceinline__ float cluster_sum(float v, float* sh, float* part, cooperative_groups::cluster_group& cl, int cs) {
+    v = block_sum(v, sh);
+    if (cs > 1) {
+        if (threadIdx.x == 0) *part = v;
+        cl.sync();
+        v = 0.0f;
+        for (int i = 0; i < cs; ++i) v += *cl.map_shared_rank(part, i);
+    }
+    return v;
+}
+
+// Columns of one row that a CTA of the cluster owns.
+struct Span { int c0, c1; };
+__device__ __forceinline__ Span cluster_span(int cols, int cs, int rank) {
+    const int per = ((cols + cs - 1) / cs + 3) / 4 * 4, c0 = min(cols, rank * per);
+    return {c0, min(cols, c0 + per)};
+}
+
+// The stream's row stays in shared memory between the residual sum and the next norm.
+template <typename T, int V>
+__global__ void __launch_bounds__(RT) sandwich_kernel(const SandwichArgs a) {
+    namespace cg = cooperative_groups;
+    extern __shared__ __align__(16) float sx[];
+    __shared__ float sh[RT / 32], part[2];
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    cg::cluster_group cl = cg::this_cluster();
+    const int cs = (int) cl.num_blocks(), rank = (int) cl.block_rank(), row = blockIdx.x / cs;
+    const Span sp = cluster_span(a.cols, cs, rank);
+    const size_t at = (size_t) row * a.cols;
+    float ss = 0.0f;
+    for (int c = sp.c0 + (int) threadIdx.x * V; c < sp.c1; c += RT * V) {
+        const Vec<V> y = ld<V>(a.y + at + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss += y.v[i] * y.v[i];
+        st<V>(sx + c - sp.c0, y);
+    }
+    const float r = 1.0f / sqrtf(cluster_sum(ss, sh, part, cl, cs) / (float) a.cols + a.eps);
+    ss = 0.0f;
+    for (int c = sp.c0 + (int) threadIdx.x * V; c < sp.c1; c += RT * V) {
+        Vec<V> x = ld<V>(a.x + at + c);
+        const Vec<V> y = ld<V>(sx + c - sp.c0), g = ld<V>(a.post + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) x.v[i] += y.v[i] * r * g.v[i];
+        if (a.add) {
+            const Vec<V> e = ld<V>(a.add + at + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) x.v[i] += e.v[i];
+        }
+        st<V>(a.x + at + c, x);
+        st<V>(sx + c - sp.c0, x);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss += x.v[i] * x.v[i];
+    }
+    if (a.pre) {
+        const float q = 1.0f / sqrtf(cluster_sum(ss, sh, part + 1, cl, cs) / (float) a.cols + a.eps);
+        for (int c = sp.c0 + (int) threadIdx.x * V; c < sp.c1; c += RT * V) {
+            Vec<V> x = ld<V>(sx + c - sp.c0);
+            const Vec<V> g = ld<V>(a.pre + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) x.v[i] = x.v[i] * q * g.v[i];
+            st_act<V>((T*) a.act + (size_t) row * a.act_ld + c, x);
+        }
+    }
+    if (cs > 1) cl.sync();                                      // no CTA leaves while its partial sums may still be read
+}
+
+// The angle is formed and reduced to one turn in double, so far positions lose nothing to its size.
+__device__ __forceinline__ float2 sin_cos_turn(double angle) {
+    angle -= rint(angle * 0.15915494309189535) * 6.283185307179586;
+    float2 r;
+    sincosf((float) angle, &r.x, &r.y);
+    return r;
+}
+template <typename T>
+__global__ void __launch_bounds__(RT) embed_pos_kernel(const EmbedPosArgs a) {
+    namespace cg = cooperative_groups;
+    extern __shared__ __align__(16) float sx[];
+    __shared__ float sh[RT / 32], part;
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    cg::cluster_group cl = cg::this_cluster();
+    const int cs = (int) cl.num_blocks(), rank = (int) cl.block_rank(), row = blockIdx.x / cs;
+    const Span sp = cluster_span(a.cols, cs, rank);                     // begins at an even column
+    const int id = min(max(a.ids[row], 0), a.vocab - 1);
+    const double pos = (double) a.map.pos_of(row);
+    const size_t at = (size_t) row * a.cols;
+    float ss = 0.0f;
+    for (int c = sp.c0 + 2 * (int) threadIdx.x; c < sp.c1; c += 2 * RT) {
+        const float2 sc = sin_cos_turn(pos * a.freq[c >> 1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            if (c + i >= sp.c1) break;
+            const float v = __bfloat162float(a.table[(size_t) id * a.ld + c + i]) * a.scale + (i ? sc.y : sc.x);
+            a.x[at + c + i] = v;
+            if (a.x0) a.x0[at + c + i] = v;
+            sx[c + i - sp.c0] = v;
+            ss += v * v;
+        }
+    }
+    const float q = 1.0f / sqrtf(cluster_sum(ss, sh, &part, cl, cs) / (float) a.cols + a.eps);
+    for (int c = sp.c0 + (int) threadIdx.x; c < sp.c1; c += RT) skd::store_act((T*) a.act + (size_t) row * a.act_ld + c, sx[c - sp.c0] * q * a.pre[c]);
+    if (cs > 1) cl.sync();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(RT) embed_rows_kernel(const bf16* __restrict__ table, int ld_, const int32_t* __restrict__ ids, int cols, int vocab,
                                                         float* __restrict__ x, float* __restrict__ state0, T* __restrict__ act, int act_ld) {
@@ -116,7 +222,7 @@ __global__ void __launch_bounds__(RT) embed_rows_kernel(const bf16* __restrict__
 }
 
 template <typename T>
-__global__ void __launch_bounds__(RT) scalar_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ index, int cols, float gain, float eps,
+__global__ void __launch_bounds__(RT) row_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ index, int cols, const float* __restrict__ gains, float gain, float eps,
                                                          T* __restrict__ act, int act_ld) {
     __shared__ float sh[RT / 32];
     skd::pdl_launch_dependents();
@@ -126,22 +232,23 @@ __global__ void __launch_bounds__(RT) scalar_norm_kernel(const float* __restrict
     for (int c = threadIdx.x; c < cols; c += RT) ss += p[c] * p[c];
     ss = block_sum(ss, sh);
     const float r = 1.0f / sqrtf(ss / (float) cols + eps) * gain;
-    for (int c = threadIdx.x; c < cols; c += RT) skd::store_act(act + (size_t) blockIdx.x * act_ld + c, p[c] * r);
+    for (int c = threadIdx.x; c < cols; c += RT) skd::store_act(act + (size_t) blockIdx.x * act_ld + c, gains ? p[c] * r * gains[c] : p[c] * r);
 }
 
-template <typename T, int V>
-int32_t run_sublayer(const SublayerArgs& a, cudaStream_t s) {
+// One cluster per row; a CTA keeps its columns of the row in dynamic shared memory.
+template <typename A>
+int32_t run_row_clusters(void (*kernel)(const A), const A& a, cudaStream_t s) {
     int cs = 1;                                                 // CTAs per row: while the machine has room and a CTA keeps 256 columns
     while (cs < 8 && a.rows * cs * 2 <= sm_count() && a.cols / (cs * 2) >= 256) cs *= 2;
     const int per = ((a.cols + cs - 1) / cs + 3) / 4 * 4;
-    SK_TRY(ensure_dynamic_smem((const void*) sublayer_kernel<T, V>, per * (int) sizeof(float)));
+    SK_TRY(ensure_dynamic_smem((const void*) kernel, per * (int) sizeof(float)));
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(a.rows * cs); cfg.blockDim = dim3(RT); cfg.dynamicSmemBytes = per * sizeof(float); cfg.stream = s;
     cudaLaunchAttribute at[2];
     at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = 1;
     at[1].id = cudaLaunchAttributeClusterDimension; at[1].val.clusterDim.x = cs; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
     cfg.attrs = at; cfg.numAttrs = 2;
-    SK_CUDA(cudaLaunchKernelEx(&cfg, sublayer_kernel<T, V>, a));
+    SK_CUDA(cudaLaunchKernelEx(&cfg, kernel, a));
     return SKAINET_CUDA_OK;
 }
 
@@ -150,8 +257,20 @@ int32_t run_sublayer(const SublayerArgs& a, cudaStream_t s) {
 int32_t launch_sublayer(const SublayerArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
     const bool vec = a.cols % 4 == 0 && a.act_ld % 4 == 0 && a.state_stride % 4 == 0;
-    if (a.f32_act) return vec ? run_sublayer<float, 4>(a, s) : run_sublayer<float, 1>(a, s);
-    return vec ? run_sublayer<bf16, 4>(a, s) : run_sublayer<bf16, 1>(a, s);
+    if (a.f32_act) return run_row_clusters(vec ? sublayer_kernel<float, 4> : sublayer_kernel<float, 1>, a, s);
+    return run_row_clusters(vec ? sublayer_kernel<bf16, 4> : sublayer_kernel<bf16, 1>, a, s);
+}
+
+int32_t launch_sandwich(const SandwichArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return SKAINET_CUDA_OK;
+    const bool vec = a.cols % 4 == 0 && a.act_ld % 4 == 0;
+    if (a.f32_act) return run_row_clusters(vec ? sandwich_kernel<float, 4> : sandwich_kernel<float, 1>, a, s);
+    return run_row_clusters(vec ? sandwich_kernel<bf16, 4> : sandwich_kernel<bf16, 1>, a, s);
+}
+
+int32_t launch_embed_pos(const EmbedPosArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return SKAINET_CUDA_OK;
+    return a.f32_act ? run_row_clusters(embed_pos_kernel<float>, a, s) : run_row_clusters(embed_pos_kernel<bf16>, a, s);
 }
 
 int32_t launch_embed_rows(const bf16* table, int ld_, const int32_t* ids, int rows, int cols, int vocab, float* x, float* state0, void* act, int act_ld,
@@ -162,10 +281,17 @@ int32_t launch_embed_rows(const bf16* table, int ld_, const int32_t* ids, int ro
     return SKAINET_CUDA_OK;
 }
 
+int32_t launch_row_norm(const float* x, const int32_t* index, int rows, int cols, const float* gain, float eps, void* act, int act_ld, bool f32_act, cudaStream_t s) {
+    if (rows <= 0) return SKAINET_CUDA_OK;
+    if (f32_act) SK_CUDA(launch_pdl(row_norm_kernel<float>, dim3(rows), dim3(RT), 0, s, x, index, cols, gain, 1.0f, eps, (float*) act, act_ld));
+    else SK_CUDA(launch_pdl(row_norm_kernel<bf16>, dim3(rows), dim3(RT), 0, s, x, index, cols, gain, 1.0f, eps, (bf16*) act, act_ld));
+    return SKAINET_CUDA_OK;
+}
+
 int32_t launch_scalar_norm(const float* x, const int32_t* index, int rows, int cols, float gain, float eps, void* act, int act_ld, bool f32_act, cudaStream_t s) {
     if (rows <= 0) return SKAINET_CUDA_OK;
-    if (f32_act) SK_CUDA(launch_pdl(scalar_norm_kernel<float>, dim3(rows), dim3(RT), 0, s, x, index, cols, gain, eps, (float*) act, act_ld));
-    else SK_CUDA(launch_pdl(scalar_norm_kernel<bf16>, dim3(rows), dim3(RT), 0, s, x, index, cols, gain, eps, (bf16*) act, act_ld));
+    if (f32_act) SK_CUDA(launch_pdl(row_norm_kernel<float>, dim3(rows), dim3(RT), 0, s, x, index, cols, (const float*) nullptr, gain, eps, (float*) act, act_ld));
+    else SK_CUDA(launch_pdl(row_norm_kernel<bf16>, dim3(rows), dim3(RT), 0, s, x, index, cols, (const float*) nullptr, gain, eps, (bf16*) act, act_ld));
     return SKAINET_CUDA_OK;
 }
 

@@ -65,7 +65,6 @@ struct Tivazen : Decoder {
     Weight *embed = nullptr, *head = nullptr;
     float final_norm = 1.0f;
     std::set<std::tuple<int, int, int>> missing;       // (layer, matrix | 100 + vector, expert) not set yet
-    std::vector<void*> owned;                          // device allocations freed with the model
     // per row in flight
     float *x = nullptr, *states = nullptr, *proj = nullptr, *gates = nullptr, *y = nullptr, *part = nullptr, *z = nullptr;
     void *act = nullptr, *act_sorted = nullptr, *act_final = nullptr;
@@ -76,17 +75,7 @@ struct Tivazen : Decoder {
         for (auto& L : layers) for (Weight* w : {L.proj, L.uk, L.uv, L.o, L.router, L.gate, L.up, L.down}) if (w) weight_release(w);
         if (embed) weight_release(embed);
         if (head) weight_release(head);
-        for (void* p : owned) cudaFree(p);
     }
-
-    // Zeroed: the tails of activation rows and cache rows are read as zeros and never written.
-    int32_t alloc(void** p, size_t bytes) {
-        SK_CUDA(cudaMalloc(p, std::max<size_t>(bytes, 16)));
-        owned.push_back(*p);
-        SK_CUDA(cudaMemset(*p, 0, std::max<size_t>(bytes, 16)));
-        return SKAINET_CUDA_OK;
-    }
-    template <typename T> int32_t alloc(T** p, size_t count) { return alloc((void**) p, count * sizeof(T)); }
 
     int32_t create(const skainet_tivazen_layer* ls);
     int32_t body(int rows, RowMap map, int kv_bound, cudaStream_t s);

@@ -1,5 +1,5 @@
 """What every model design of libskainet_cuda's decoder runtime offers to a host (include/skainet_cuda_llama.h): sequence slots,
-prompts, single decode steps, logits of chosen positions, greedy generation. The designs (llama.py, tivazen.py) add how a
+prompts, single decode steps, logits of chosen positions, greedy generation. The designs (llama.py, tivazen.py, fomalix.py) add how a
 model is configured and loaded."""
 from __future__ import annotations
 
@@ -85,7 +85,7 @@ class Decoder:
 
     def peek(self, which: int, n: int) -> np.ndarray:
         """Diagnostic read of an activation buffer; what `which` names is the design's (Llama: 0 x, 1 q|k|v, 2 attention out,
-        3 gate|up, 4 q; Tivazen: 0 x, 1 merged projection, 16 + j the state X_j of the rows last run)."""
+        3 gate|up, 4 q; Tivazen: 0 x, 1 merged projection, 16 + j the state X_j of the rows last run; Fomalix: 0 x, 1 merged projection)."""
         out = np.empty(n, dtype=np.float32)
         L.check(L.lib().skainet_cuda_llama_peek(self.handle, which, out.ctypes.data_as(L.f32p), n))
         return out

@@ -12,10 +12,11 @@ import os
 from typing import Callable, Dict, List, Sequence
 
 from .decoder import Decoder
+from .fomalix import Fomalix
 from .llama import Llama
 from .tivazen import Tivazen
 
-FOLDERS: Dict[str, Callable[..., Decoder]] = {Tivazen.architecture: Tivazen.from_dir}
+FOLDERS: Dict[str, Callable[..., Decoder]] = {Tivazen.architecture: Tivazen.from_dir, Fomalix.architecture: Fomalix.from_dir}
 GGUF: Dict[str, Callable[..., Decoder]] = {"llama": Llama.from_gguf}
 
 
