@@ -30,6 +30,9 @@ Prints ONE JSON line (rank 0). Workloads (all inputs synthetic and seeded):
       in a CUDA graph: the peer-memory sum, the store + gather + sum + RMSNorm + quantize kernel, and ncclAllReduce of the
       same row; metric = microseconds per exchange (lower is better). The N > 1 decode lines carry the same three numbers
       under `tp_exchange`.
+  fomalix — the Fomalix design at --size (7b, 2b: random weights in the shape of a real model's layers) beside the Tivazen model
+      of the same layer count, width, heads and inner size: greedy decode steps behind --context positions and a --prompt-token
+      prefill of each; metric = the Fomalix model's decode tokens/s. One GPU.
   tivazen — the Tivazen design at --size (7b, 2b, moe: random weights in the shape of a real model's layers) beside a Llama-style
       Q4_K model of the same layers, width, heads and inner size: greedy decode of --batch sequences behind a --context window
       and a --prompt-token prefill of each; metric = the Tivazen model's decode tokens/s. One GPU.
@@ -264,8 +267,8 @@ def run_reference(args) -> None:
     rank, _, _ = dist_env()
     if rank != 0:
         return
-    if args.workload == "tivazen":
-        print(json.dumps({"impl": "reference", "unavailable": "the reference has no Tivazen model"}), flush=True)
+    if args.workload in ("tivazen", "fomalix"):
+        print(json.dumps({"impl": "reference", "unavailable": f"the reference has no {args.workload.capitalize()} model"}), flush=True)
         return
     budget = max(2.0, min(20.0, 90.0 / max(1, args.steps + args.warmup)))
     vals, times = [], []
@@ -995,6 +998,82 @@ def run_tivazen(args) -> None:
     print(json.dumps(line), flush=True)
 
 
+FOMALIX_SIZES = {
+    # layers, width, (attention heads, key/value heads, chunk), (delta-rule heads, query/key heads), (Mamba-2 heads x 64, groups), ff, vocab
+    "7b": (32, 4096, (32, 8, 8192), (32, 16), (128, 8), 11008, 32000),
+    "2b": (24, 2048, (16, 4, 2048), (16, 8), (64, 4), 5632, 32000),
+}
+
+
+def fomalix_config(size: str, **kw):
+    """Layers in turns of four: two of the delta rule, one Mamba-2, one attention, each with a feed-forward; heads of 128."""
+    from skainet_b200.fomalix import ATTENTION, DELTA, MAMBA2, FomalixConfig, FomalixLayer
+    n, width, (ah, akv, chunk), (dh, dqk), (mh, mg), ff, vocab = FOMALIX_SIZES[size]
+    turn = [FomalixLayer(DELTA, dh, dqk, 128, 128, conv=4, ff=ff)] * 2 + [FomalixLayer(MAMBA2, mh, mg, 128, 64, conv=4, norm_groups=1, ff=ff),
+                                                                       FomalixLayer(ATTENTION, ah, akv, 128, 128, chunk=chunk, scale=1.0, ff=ff)]
+    return FomalixConfig(width, vocab, 1e-5, (turn * n)[:n], 12.0, **kw)
+
+
+def fomalix_linear_flops(cfg) -> float:
+    """Multiply-adds x 2 of the linears per prompt token (attention and recurrences come on top)."""
+    from skainet_b200.fomalix import ATTENTION, DELTA
+    total = 0
+    for l in cfg.layers:
+        qk, inner = l.kv_heads * l.dim, l.heads * l.vdim
+        rows = {ATTENTION: l.heads * l.dim + qk + l.kv_heads * l.vdim, DELTA: 2 * qk + 2 * inner + 2 * l.heads}.get(l.type, 2 * inner + 2 * qk + l.heads)
+        total += cfg.width * (rows + inner + 3 * l.ff)
+    return 2.0 * total
+
+
+def run_fomalix(args) -> None:
+    import torch
+    from skainet_b200 import _lib as L, device
+    from skainet_b200.fomalix import Fomalix
+    from skainet_b200.tivazen import MLP_DENSE, Tivazen, TivazenConfig, TivazenLayer
+    rank, world, local = dist_env()
+    torch.cuda.set_device(local); device.set_device(local)
+    size = args.size if args.size in FOMALIX_SIZES else "7b"
+    n, width, (heads, _, chunk), _, _, ff, vocab = FOMALIX_SIZES[size]
+    batch, n_prompt, warm = max(1, args.batch), args.prompt, max(3, args.warmup)
+    ctx = min(args.context, chunk - args.steps - warm - 8)
+    room = max(ctx + args.steps + warm + 8, n_prompt)
+    sampler = ClockSampler(local); sampler.start()
+    cfg = fomalix_config(size, max_seq=room, max_batch=batch)
+    m = Fomalix(cfg)
+    m.synth(seed=100, std=0.02)
+    m.finalize()
+    ours = decoder_phases(torch, m, batch, ctx, n_prompt, args.steps, warm, vocab)
+    m.free()
+    near = None
+    if not args.skip_cpu:
+        near_cfg = TivazenConfig(width, vocab, 1e-5, [TivazenLayer(heads, 128, 64, 128, 512, chunk, (128 + 64) ** -0.5, 1e4, None, MLP_DENSE, ff)] * n, max_seq=room, max_batch=batch)
+        k = Tivazen(near_cfg)
+        k.synth(seed=100, std=0.02)
+        k.finalize()
+        near = decoder_phases(torch, k, batch, ctx, n_prompt, args.steps, warm, vocab)
+        k.free()
+    clocks = sampler.stop()
+    if L.lib().skainet_cuda_device_status() != 0:
+        raise SystemExit(f"device error: {L.last_error()}")
+    peak, peak_kind = load_peaks()
+    tpeak, _ = load_tensor_peak()
+    for d, flops in ((ours, fomalix_linear_flops(cfg)),) + (((near, tivazen_linear_flops(near_cfg)),) if near else ()):
+        d["prefill_linear_tflops"] = flops * n_prompt / d["prefill_ms"] / 1e9
+        d["prefill_frac_of_bf16_burst"] = d["prefill_linear_tflops"] / tpeak
+        d["decode_frac"] = d["decode_gbs"] / peak
+    line = {"metric": "fomalix_decode_tokens_per_s", "value": ours["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": warm,
+            "ms_per_step": ours["decode_ms"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+            "dtype": "bf16 weights, activations and cache, f32 accumulate (residual, norms, scores, recurrences and their state f32)", "data": "synthetic",
+            "config": {"workload": "fomalix", "size": size, "layers": n, "width": width, "turn": "delta, delta, mamba2, attention", "heads": heads, "chunk": chunk, "ff": ff, "vocab": vocab,
+                       "batch": batch, "context": ctx, "context_fill": "seeded noise", "prompt_tokens": n_prompt, "weights": "N(0,0.02), seeded",
+                       "l2": "weights per step far larger than L2", "parallelism": "single"},
+            "roofline": {"bound": "hbm", "achieved": ours["decode_gbs"], "peak": peak, "unit": "GB/s", "frac": ours["decode_gbs"] / peak, "traffic": None,
+                         "peak_kind": peak_kind, "kernel": "whole decode step"},
+            "fomalix": ours, "closest_tivazen": near, "gpu_launches": ours["launches_per_step"] * args.steps, "clocks": clocks,
+            "e2e": {"value": batch / ours["e2e_ms"] * 1e3, "unit": "tokens/s", "h2d_bytes_per_step": 4 * batch, "d2h_bytes_per_step": 4 * batch}}
+    print(json.dumps(line), flush=True)
+
+
 def run_kv_turboquant(args) -> None:
     """kv_turboquant: the TurboQuant KV store (4-bit keys and values, 8 heads x 128) behind one decode step of attention over
     --context positions: decode of the window's blocks to fp32 + fp32 attention, per layer of a 32-layer store (the layers'
@@ -1282,13 +1361,13 @@ def main() -> None:
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=5)
-    ap.add_argument("--workload", default="decode_70b", choices=sorted(MATVEC_WORKLOADS) + sorted(DECODE_WORKLOADS) + sorted(ATTN_WORKLOADS) + sorted(GEMM_WORKLOADS) + sorted(REQUEST_WORKLOADS) + ["tivazen", "tp_collective", "kv_turboquant"])
-    ap.add_argument("--context", type=int, default=4096, help="keys per sequence (attn_decode, tivazen workloads)")
+    ap.add_argument("--workload", default="decode_70b", choices=sorted(MATVEC_WORKLOADS) + sorted(DECODE_WORKLOADS) + sorted(ATTN_WORKLOADS) + sorted(GEMM_WORKLOADS) + sorted(REQUEST_WORKLOADS) + ["tivazen", "fomalix", "tp_collective", "kv_turboquant"])
+    ap.add_argument("--context", type=int, default=4096, help="keys per sequence (attn_decode, tivazen, fomalix workloads)")
     ap.add_argument("--batch", type=int, default=1, help="sequences decoded together (decode workloads)")
-    ap.add_argument("--size", default="7b", choices=sorted(TIVAZEN_SIZES), help="model shape of the tivazen workload")
-    ap.add_argument("--prompt", type=int, default=2048, help="prompt tokens of the tivazen workload's prefill")
+    ap.add_argument("--size", default="7b", choices=sorted(TIVAZEN_SIZES), help="model shape of the tivazen and fomalix workloads")
+    ap.add_argument("--prompt", type=int, default=2048, help="prompt tokens of the tivazen and fomalix workloads' prefill")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--skip-cpu", action="store_true", help="omit the cpu_baseline leg, or the Llama-style comparison of the tivazen workload (profiling runs)")
+    ap.add_argument("--skip-cpu", action="store_true", help="omit the cpu_baseline leg, or the comparison model of the tivazen and fomalix workloads (profiling runs)")
     ap.add_argument("--skip-e2e", action="store_true", help="omit the end-to-end leg (profiling runs)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -1305,6 +1384,8 @@ def main() -> None:
         run_collective(args)
     elif args.workload == "tivazen":
         run_tivazen(args)
+    elif args.workload == "fomalix":
+        run_fomalix(args)
     elif args.workload == "kv_turboquant":
         run_kv_turboquant(args)
     else:
