@@ -1,6 +1,10 @@
 // Ring attention with a chunk mask and a sink (contract: kv_attn.cuh).
 //
 //   kv_prep_kernel       biases, unit-rms queries and keys, ring append.
+//   kv_attn_tile_kernel  bf16: the MMA rows are (activation row, head) pairs that share a key/value head, so a staged key or value
+//                        row serves the whole group. In prompts each of eight warps owns 16 pairs and all read the same tile of 64
+//                        keys; in a decode step four warps own the same 16 pairs and a quarter of the tile's keys each. Keys may
+//                        be split over CTAs; kv_merge_kernel joins the parts in fixed order.
 //   kv_attn_rows_kernel  fp32 FMA, one CTA per (row, head), any size: the 32-bit mode, and bf16 models whose heads are too large
 //                        for the tile kernel.
 #include "kv_attn.cuh"
@@ -99,6 +103,275 @@ __global__ void __launch_bounds__(RK) kv_attn_rows_kernel(const KvAttnArgs a) {
     for (int d = t; d < g.vdim; d += RK) skd::store_act((T*) a.out + (size_t) row * g.out_ld() + h * g.vdim + d, acc[d] / l);
 }
 
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int TK = 64;                       // keys of a staged tile
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// Widths up to 16 * KS (keys) and 8 * VN (values). DECODE: the activation rows of a CTA are one, its warps split the keys.
+template <int KS, int VN, bool DECODE>
+struct TileShape {
+    static constexpr int WARPS = DECODE ? 4 : 8, ROWS = DECODE ? 16 : 128, KEYS = DECODE ? TK / WARPS : TK;   // pairs of a CTA, keys of a warp
+    static constexpr int STAGES = DECODE ? 3 : 2;
+    static constexpr bool Q_REGS = KS <= 8;
+    // rows are 16 bytes longer than the data: an odd number of 16-byte units, so ldmatrix rows meet different banks
+    static __host__ __device__ int smem(int kld, int vcld) {
+        const int tiles = (ROWS * (kld + 8) + STAGES * TK * (kld + 8 + vcld + 8)) * 2, merge = DECODE ? WARPS * 16 * (vcld + 2) * 4 : 0;
+        return tiles > merge ? tiles : merge;
+    }
+};
+
+template <int KS, int VN, bool DECODE>
+__global__ void __launch_bounds__(TileShape<KS, VN, DECODE>::WARPS * 32)
+kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
+    typedef TileShape<KS, VN, DECODE> S;
+    extern __shared__ __align__(16) uint8_t raw[];
+    const KvGeom g = a.g;
+    const int kld = g.kld(), vcld = g.vcld(), klds = kld + 8, vlds = vcld + 8, ks_n = kld / 16, vn_n = vcld / 8;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, tq = lane & 3, group = g.heads / g.kv_heads;
+    const int kh = blockIdx.y, split = blockIdx.z;
+    // pairs [p0, p0 + ROWS) of this key/value head: row p / group, head p % group
+    const int tiles_m = DECODE ? (group + 15) / 16 : 0;
+    const int m_tile = DECODE ? (int) blockIdx.x % tiles_m : (int) (gridDim.x - 1 - blockIdx.x);          // the longest prompt tiles first
+    const int row_base = DECODE ? (int) blockIdx.x / tiles_m : 0, p0 = m_tile * S::ROWS, pairs = DECODE ? group : a.rows * group;
+    const uint32_t sq = skd::smem_u32(raw), sk = sq + S::ROWS * klds * 2, sv = sk + S::STAGES * TK * klds * 2;
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    const int seq = a.map.seq_of(row_base);
+    const bf16* kc = (const bf16*) a.cache.k + ((size_t) seq * g.kv_heads + kh) * a.cache.cap * kld;
+    const bf16* vc = (const bf16*) a.cache.v + ((size_t) seq * g.kv_heads + kh) * a.cache.cap * vcld;
+    const int first_row = row_base + p0 / group, last_row = row_base + (min(pairs, p0 + S::ROWS) - 1) / group;
+    const int pos_first = a.map.pos_of(first_row), pos_last = a.map.pos_of(last_row);
+    const int lo = first_key(a, pos_first), lo_last = first_key(a, pos_last);
+    int t0 = 0, t1 = (pos_last - lo) / TK + 1;
+    if (splits > 1) { const int per = (t1 + splits - 1) / splits; t0 = min(t1, split * per); t1 = min(t1, t0 + per); }
+
+    auto load_tile = [&](int t, int stage) {
+        const int j0 = lo + t * TK, kch = kld / 8, vch = vcld / 8, slot0 = j0 % a.cache.cap;
+        for (int i = threadIdx.x; i < TK * (kch + vch); i += S::WARPS * 32) {
+            const bool is_v = i >= TK * kch;
+            const int e = is_v ? i - TK * kch : i, ch = is_v ? vch : kch, r = e / ch, c = e % ch;
+            int slot = slot0 + r;
+            if (slot >= a.cache.cap) slot %= a.cache.cap;
+            if (is_v) cp16(sv + ((stage * TK + r) * vlds + c * 8) * 2, vc + (size_t) slot * vcld + c * 8);
+            else cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
+        }
+    };
+    // queries; rows past the last pair repeat it and are not stored
+    for (int i = threadIdx.x; i < S::ROWS * (kld / 8); i += S::WARPS * 32) {
+        const int r = i / (kld / 8), c = i % (kld / 8), p = min(p0 + r, pairs - 1);
+        cp16(sq + (r * klds + c * 8) * 2, (const bf16*) a.q + ((size_t) (row_base + p / group) * g.heads + kh * group + p % group) * kld + c * 8);
+    }
+#pragma unroll
+    for (int s = 0; s < S::STAGES - 1; ++s) { if (t0 + s < t1) load_tile(t0 + s, s); cp_commit(); }
+
+    const int wr = DECODE ? 0 : warp * 16;                        // the warp's first pair
+    int pos_r[2], lo_r[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        pos_r[i] = a.map.pos_of(row_base + min(p0 + wr + gr + 8 * i, pairs - 1) / group);
+        lo_r[i] = first_key(a, pos_r[i]);
+    }
+    float o[VN][4];
+#pragma unroll
+    for (int n = 0; n < VN; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[n][i] = 0.0f;
+    float m[2] = {NEG_BIG, NEG_BIG}, l[2] = {0.0f, 0.0f};
+    uint32_t qf[S::Q_REGS ? KS : 1][4];
+    const uint32_t q_at = sq + ((wr + (lane & 7) + ((lane >> 3) & 1) * 8) * klds + (lane >> 4) * 8) * 2;
+    const int k0w = DECODE ? warp * S::KEYS : 0;                  // the warp's first key of a tile
+    const uint32_t k_at = sk + ((k0w + (lane & 7) + (lane >> 4) * 8) * klds + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t v_at = sv + ((k0w + (lane & 7) + ((lane >> 3) & 1) * 8) * vlds + (lane >> 4) * 8) * 2;
+    const float sc2 = a.scale * LOG2E;
+    constexpr int NK = S::KEYS / 8;
+
+    for (int t = t0; t < t1; ++t) {
+        const int stage = (t - t0) % S::STAGES;
+        cp_wait<S::STAGES - 2>();
+        __syncthreads();
+        if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES);
+        cp_commit();
+        if (S::Q_REGS && t == t0)
+#pragma unroll
+            for (int k = 0; k < KS; ++k) if (k < ks_n) ldsm4(qf[S::Q_REGS ? k : 0], q_at + k * 32);
+        float c[NK][4];
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) c[n][i] = 0.0f;
+#pragma unroll
+        for (int k = 0; k < KS; ++k) {
+            if (k >= ks_n) break;
+            uint32_t qk[4];
+            if (!S::Q_REGS) ldsm4(qk, q_at + k * 32);
+            const uint32_t* q = S::Q_REGS ? qf[S::Q_REGS ? k : 0] : qk;
+#pragma unroll
+            for (int n = 0; n < NK; n += 2) {
+                uint32_t b[4];
+                ldsm4(b, k_at + ((stage * TK + n * 8) * klds + k * 16) * 2);
+                skd::mma_bf16(c[n], q[0], q[1], q[2], q[3], b[0], b[1]);
+                skd::mma_bf16(c[n + 1], q[0], q[1], q[2], q[3], b[2], b[3]);
+            }
+        }
+        const int j0 = lo + t * TK + k0w;
+        const bool whole = j0 >= lo_last && j0 + S::KEYS - 1 <= pos_first;
+        float mx[2] = {m[0], m[1]};
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int j = j0 + n * 8 + tq * 2 + (i & 1);
+                c[n][i] = whole || (j >= lo_r[i >> 1] && j <= pos_r[i >> 1]) ? c[n][i] * sc2 : -INFINITY;
+                mx[i >> 1] = fmaxf(mx[i >> 1], c[n][i]);
+            }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(~0u, mx[i], 1)); mx[i] = fmaxf(mx[i], __shfl_xor_sync(~0u, mx[i], 2));
+            const float fade = exp2f(m[i] - mx[i]);
+            m[i] = mx[i];
+            l[i] *= fade;
+            if (__any_sync(~0u, fade != 1.0f))
+#pragma unroll
+                for (int n = 0; n < VN; ++n) { o[n][2 * i] *= fade; o[n][2 * i + 1] *= fade; }
+        }
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { c[n][i] = exp2f(c[n][i] - m[i >> 1]); l[i >> 1] += c[n][i]; }
+#pragma unroll
+        for (int k = 0; k < NK / 2; ++k) {
+            const uint32_t p[4] = {skd::pack_bf16(c[2 * k][0], c[2 * k][1]), skd::pack_bf16(c[2 * k][2], c[2 * k][3]), skd::pack_bf16(c[2 * k + 1][0], c[2 * k + 1][1]),
+                                   skd::pack_bf16(c[2 * k + 1][2], c[2 * k + 1][3])};
+#pragma unroll
+            for (int n = 0; n < VN; n += 2) {
+                if (n >= vn_n) break;
+                uint32_t b[4];
+                ldsm4_t(b, v_at + ((stage * TK + k * 16) * vlds + n * 8) * 2);
+                skd::mma_bf16(o[n], p[0], p[1], p[2], p[3], b[0], b[1]);
+                skd::mma_bf16(o[n + 1], p[0], p[1], p[2], p[3], b[2], b[3]);
+            }
+        }
+    }
+    cp_wait<0>();                                                 // the queries of a part without keys are still in flight
+#pragma unroll
+    for (int i = 0; i < 2; ++i) { l[i] += __shfl_xor_sync(~0u, l[i], 1); l[i] += __shfl_xor_sync(~0u, l[i], 2); }
+
+    // Joins the sink, or leaves a record. `w` writes one pair's columns.
+    auto finish = [&](int p, float mm, float ll, auto&& value, int d_first, int d_step, bool lead) {
+        if (p >= pairs) return;
+        const int row = row_base + p / group, h = kh * group + p % group;
+        if (splits > 1) {
+            float* rec = a.part + (((size_t) row * g.heads + h) * splits + split) * (vcld + 2);
+            for (int d = d_first; d < vcld; d += d_step) value(d, [&](int at, float v) { rec[at] = v; });
+            if (lead) { rec[vcld] = mm; rec[vcld + 1] = ll; }
+            return;
+        }
+        float f = 1.0f, den = ll;
+        if (a.sink) {
+            const float s2 = a.sink[h] * LOG2E, top = fmaxf(mm, s2);
+            f = exp2f(mm - top);
+            den = ll * f + exp2f(s2 - top);
+        }
+        f /= den;
+        bf16* out = (bf16*) a.out + (size_t) row * g.out_ld() + h * g.vdim;
+        for (int d = d_first; d < g.vdim; d += d_step) value(d, [&](int at, float v) { if (at < g.vdim) out[at] = __float2bfloat16_rn(v * f); });
+    };
+    if (!DECODE) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+            finish(p0 + wr + gr + 8 * i, m[i], l[i], [&](int d, auto&& put) {
+                (void) d;
+#pragma unroll
+                for (int n = 0; n < VN; ++n) if (n < vn_n) { put(n * 8 + tq * 2, o[n][2 * i]); put(n * 8 + tq * 2 + 1, o[n][2 * i + 1]); }
+            }, 0, 1 << 20, tq == 0);
+    } else {
+        // the warps' parts meet in shared memory: [warp][pair][vcld + 2]
+        float* part = (float*) raw;
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            float* rec = part + (warp * 16 + gr + 8 * i) * (vcld + 2);
+#pragma unroll
+            for (int n = 0; n < VN; ++n) if (n < vn_n) { rec[n * 8 + tq * 2] = o[n][2 * i]; rec[n * 8 + tq * 2 + 1] = o[n][2 * i + 1]; }
+            if (tq == 0) { rec[vcld] = m[i]; rec[vcld + 1] = l[i]; }
+        }
+        __syncthreads();
+        for (int r = warp; r < 16 && p0 + r < pairs; r += S::WARPS) {
+            float top = NEG_BIG, sum = 0.0f, f[S::WARPS];
+#pragma unroll
+            for (int w = 0; w < S::WARPS; ++w) top = fmaxf(top, part[(w * 16 + r) * (vcld + 2) + vcld]);
+#pragma unroll
+            for (int w = 0; w < S::WARPS; ++w) {
+                const float* rec = part + (w * 16 + r) * (vcld + 2) + vcld;
+                f[w] = exp2f(rec[0] - top);
+                sum += rec[1] * f[w];
+            }
+            finish(p0 + r, top, sum, [&](int d, auto&& put) {
+                float v = 0.0f;
+#pragma unroll
+                for (int w = 0; w < S::WARPS; ++w) v += part[(w * 16 + r) * (vcld + 2) + d] * f[w];
+                put(d, v);
+            }, lane, 32, lane == 0);
+        }
+    }
+}
+
+// One warp per (row, head): the records of the splits, then the sink.
+__global__ void __launch_bounds__(128) kv_merge_kernel(const KvAttnArgs a, int splits) {
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    const KvGeom& g = a.g;
+    const int h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, row = blockIdx.x, ld = g.vcld() + 2;
+    if (h >= g.heads) return;
+    const float* rec = a.part + ((size_t) row * g.heads + h) * splits * ld;
+    float top = NEG_BIG;
+    for (int s = lane; s < splits; s += 32) top = fmaxf(top, rec[(size_t) s * ld + g.vcld()]);
+    top = skd::warp_max(top);
+    float den = 0.0f;
+    if (a.sink) { const float s2 = a.sink[h] * LOG2E; top = fmaxf(top, s2); den = exp2f(s2 - top); }
+    for (int s = 0; s < splits; ++s) den += rec[(size_t) s * ld + g.vcld() + 1] * exp2f(rec[(size_t) s * ld + g.vcld()] - top);
+    for (int d = lane; d < g.vdim; d += 32) {
+        float v = 0.0f;
+#pragma unroll 4
+        for (int s = 0; s < splits; ++s) v = fmaf(rec[(size_t) s * ld + d], exp2f(rec[(size_t) s * ld + g.vcld()] - top), v);
+        ((bf16*) a.out)[(size_t) row * g.out_ld() + h * g.vdim + d] = __float2bfloat16_rn(v / den);
+    }
+}
+
+// Pairs of a step's row reach no further than one row, so a decode step has a CTA row per sequence; prompts tile the pairs.
+template <int KS, int VN, bool DECODE>
+int32_t run_tile(const KvAttnArgs& a, cudaStream_t s) {
+    typedef TileShape<KS, VN, DECODE> S;
+    const KvGeom& g = a.g;
+    const int group = g.heads / g.kv_heads, bytes = S::smem(g.kld(), g.vcld());
+    const int mx = DECODE ? a.rows * ((group + 15) / 16) : (a.rows * group + S::ROWS - 1) / S::ROWS;
+    const int seen = a.chunk > 0 ? std::min(a.kv_bound, a.chunk + (DECODE ? 0 : a.rows)) : a.kv_bound;
+    const int64_t room = (int64_t) KV_PART_RECORDS / ((int64_t) a.rows * g.heads);
+    const int want = (2 * sm_count() + mx * g.kv_heads - 1) / (mx * g.kv_heads);
+    int splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) want, (int64_t) (seen + TK - 1) / TK, room, 65535}));
+    if (!DECODE && mx * g.kv_heads * 2 > sm_count()) splits = 1;
+    SK_TRY(ensure_dynamic_smem((const void*) kv_attn_tile_kernel<KS, VN, DECODE>, bytes));
+    SK_CUDA(launch_pdl(kv_attn_tile_kernel<KS, VN, DECODE>, dim3(mx, g.kv_heads, splits), dim3(S::WARPS * 32), bytes, s, a, splits));
+    if (splits > 1) SK_CUDA(launch_pdl(kv_merge_kernel, dim3(a.rows, (g.heads + 3) / 4), dim3(128), 0, s, a, splits));
+    return SKAINET_CUDA_OK;
+}
+template <bool DECODE>
+int32_t run_tile_size(const KvAttnArgs& a, cudaStream_t s) {
+    const int n = std::max(a.g.kld(), a.g.vcld());
+    if (n <= 64) return run_tile<4, 8, DECODE>(a, s);
+    if (n <= 128) return run_tile<8, 16, DECODE>(a, s);
+    return run_tile<16, 32, DECODE>(a, s);
+}
+
 template <typename T>
 int32_t run_rows(const KvAttnArgs& a, cudaStream_t s) {
     const int bytes = (a.g.kld() + a.g.vcld()) * (int) sizeof(float);
@@ -114,13 +387,12 @@ int32_t run_prep(const KvAttnArgs& a, cudaStream_t s) {
 
 }  // namespace
 
-size_t kv_part_floats(const KvGeom& g) { (void) g; return 0; }
-
 int32_t launch_kv_attention(const KvAttnArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
     if (a.f32_act) { SK_TRY(run_prep<float>(a, s)); return run_rows<float>(a, s); }
     SK_TRY(run_prep<bf16>(a, s));
-    return run_rows<bf16>(a, s);
+    if (a.g.kld() > 256 || a.g.vcld() > 256) return run_rows<bf16>(a, s);
+    return a.map.seq < 0 ? run_tile_size<true>(a, s) : run_tile_size<false>(a, s);
 }
 
 }  // namespace sk

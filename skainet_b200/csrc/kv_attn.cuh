@@ -33,15 +33,15 @@ struct KvAttnArgs {
     const float *sink = nullptr;          // [heads], or null
     KvCache cache;
     void *q = nullptr, *out = nullptr;    // activation type: prepared queries [row][head][kld]; concatenated heads [row][out_ld]
-    float* part = nullptr;                // key-split records, kv_part_floats() of them
+    float* part = nullptr;                // key-split records, kv_part_floats() floats
     int rows = 0;
     RowMap map = {nullptr, -1};
     int kv_bound = 0;                     // bound on the sequence length after this step
     bool f32_act = false;
 };
 
-// Floats of KvAttnArgs::part.
-size_t kv_part_floats(const KvGeom& g);
+constexpr int KV_PART_RECORDS = 64 * 320;   // (row, head, split) records a split launch may use: [mixed values, vcld | maximum | sum]
+inline size_t kv_part_floats(const KvGeom& g) { return (size_t) KV_PART_RECORDS * (g.vcld() + 2); }
 
 // proj -> biases, norms, ring append, attention, concatenated heads in a.out.
 int32_t launch_kv_attention(const KvAttnArgs& a, cudaStream_t s);
