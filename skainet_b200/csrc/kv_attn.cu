@@ -8,6 +8,7 @@
 //   kv_attn_rows_kernel  fp32 FMA, one CTA per (row, head), any size: the 32-bit mode, and bf16 models whose heads are too large
 //                        for the tile kernel.
 #include "kv_attn.cuh"
+#include "mma.cuh"
 #include "tma.cuh"
 
 #include <algorithm>
@@ -106,16 +107,6 @@ __global__ void __launch_bounds__(RK) kv_attn_rows_kernel(const KvAttnArgs a) {
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int TK = 64;                       // keys of a staged tile
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 // Widths up to 16 * KS (keys) and 8 * VN (values). DECODE: the activation rows of a CTA are one, its warps split the keys.
 template <int KS, int VN, bool DECODE>
 struct TileShape {
@@ -161,17 +152,17 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
             const int e = is_v ? i - TK * kch : i, ch = is_v ? vch : kch, r = e / ch, c = e % ch;
             int slot = slot0 + r;
             if (slot >= a.cache.cap) slot %= a.cache.cap;
-            if (is_v) cp16(sv + ((stage * TK + r) * vlds + c * 8) * 2, vc + (size_t) slot * vcld + c * 8);
-            else cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
+            if (is_v) skd::cp16(sv + ((stage * TK + r) * vlds + c * 8) * 2, vc + (size_t) slot * vcld + c * 8);
+            else skd::cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
         }
     };
     // queries; rows past the last pair repeat it and are not stored
     for (int i = threadIdx.x; i < S::ROWS * (kld / 8); i += S::WARPS * 32) {
         const int r = i / (kld / 8), c = i % (kld / 8), p = min(p0 + r, pairs - 1);
-        cp16(sq + (r * klds + c * 8) * 2, (const bf16*) a.q + ((size_t) (row_base + p / group) * g.heads + kh * group + p % group) * kld + c * 8);
+        skd::cp16(sq + (r * klds + c * 8) * 2, (const bf16*) a.q + ((size_t) (row_base + p / group) * g.heads + kh * group + p % group) * kld + c * 8);
     }
 #pragma unroll
-    for (int s = 0; s < S::STAGES - 1; ++s) { if (t0 + s < t1) load_tile(t0 + s, s); cp_commit(); }
+    for (int s = 0; s < S::STAGES - 1; ++s) { if (t0 + s < t1) load_tile(t0 + s, s); skd::cp_commit(); }
 
     const int wr = DECODE ? 0 : warp * 16;                        // the warp's first pair
     int pos_r[2], lo_r[2];
@@ -196,13 +187,13 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
 
     for (int t = t0; t < t1; ++t) {
         const int stage = (t - t0) % S::STAGES;
-        cp_wait<S::STAGES - 2>();
+        skd::cp_wait<S::STAGES - 2>();
         __syncthreads();
         if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES);
-        cp_commit();
+        skd::cp_commit();
         if (S::Q_REGS && t == t0)
 #pragma unroll
-            for (int k = 0; k < KS; ++k) if (k < ks_n) ldsm4(qf[S::Q_REGS ? k : 0], q_at + k * 32);
+            for (int k = 0; k < KS; ++k) if (k < ks_n) skd::ldsm4(qf[S::Q_REGS ? k : 0], q_at + k * 32);
         float c[NK][4];
 #pragma unroll
         for (int n = 0; n < NK; ++n)
@@ -212,12 +203,12 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
         for (int k = 0; k < KS; ++k) {
             if (k >= ks_n) break;
             uint32_t qk[4];
-            if (!S::Q_REGS) ldsm4(qk, q_at + k * 32);
+            if (!S::Q_REGS) skd::ldsm4(qk, q_at + k * 32);
             const uint32_t* q = S::Q_REGS ? qf[S::Q_REGS ? k : 0] : qk;
 #pragma unroll
             for (int n = 0; n < NK; n += 2) {
                 uint32_t b[4];
-                ldsm4(b, k_at + ((stage * TK + n * 8) * klds + k * 16) * 2);
+                skd::ldsm4(b, k_at + ((stage * TK + n * 8) * klds + k * 16) * 2);
                 skd::mma_bf16(c[n], q[0], q[1], q[2], q[3], b[0], b[1]);
                 skd::mma_bf16(c[n + 1], q[0], q[1], q[2], q[3], b[2], b[3]);
             }
@@ -255,13 +246,13 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
             for (int n = 0; n < VN; n += 2) {
                 if (n >= vn_n) break;
                 uint32_t b[4];
-                ldsm4_t(b, v_at + ((stage * TK + k * 16) * vlds + n * 8) * 2);
+                skd::ldsm4_t(b, v_at + ((stage * TK + k * 16) * vlds + n * 8) * 2);
                 skd::mma_bf16(o[n], p[0], p[1], p[2], p[3], b[0], b[1]);
                 skd::mma_bf16(o[n + 1], p[0], p[1], p[2], p[3], b[2], b[3]);
             }
         }
     }
-    cp_wait<0>();                                                 // the queries of a part without keys are still in flight
+    skd::cp_wait<0>();                                                 // the queries of a part without keys are still in flight
 #pragma unroll
     for (int i = 0; i < 2; ++i) { l[i] += __shfl_xor_sync(~0u, l[i], 1); l[i] += __shfl_xor_sync(~0u, l[i], 2); }
 

@@ -3,6 +3,7 @@
 //   recur_step_kernel    one token of each sequence, or consecutive tokens of one: a CTA keeps 32 columns of a head's state in
 //                        registers (columns of the state never meet), so a step reads and writes the state once.
 //   recur_tail_kernel    the convolution inputs a prompt pass leaves for the next one.
+//   recurrence_chunk.cu  prompts of bf16 models: chunks of 64 tokens on the tensor cores.
 //   gated_norm_kernel    norm and output gate.
 #include "recurrence.cuh"
 #include "tma.cuh"
@@ -15,14 +16,9 @@ namespace {
 
 constexpr int ST = 256, SC = 32;                 // threads and state columns of a step CTA
 
-__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+using skd::conv_input;
+using skd::softplus;
 
-// Input of convolution channel c at position p; rows of the pass start at position pos0 in row row0.
-__device__ __forceinline__ float conv_input(const RecurArgs& a, const float* tail, int row0, int pos0, int p, int c) {
-    if (p < 0) return 0.0f;
-    if (p >= pos0) return a.proj[(size_t) (row0 + p - pos0) * a.proj_ld + a.conv_off + c];
-    return tail[(size_t) (p % a.g.taps) * a.g.conv_dim() + c];
-}
 __device__ __forceinline__ float conv_silu(const RecurArgs& a, const float* tail, int row0, int pos0, int p, int c) {
     float v = a.conv_b ? a.conv_b[c] : 0.0f;
     for (int j = 0; j < a.g.taps; ++j) v = fmaf(a.conv_w[(size_t) c * a.g.taps + j], conv_input(a, tail, row0, pos0, p - (a.g.taps - 1) + j, c), v);
@@ -195,11 +191,10 @@ int32_t run_gated_norm(const GatedNormArgs& a, cudaStream_t s) {
 
 }  // namespace
 
-size_t recur_work_bytes(const RecurGeom& g, int rows) { (void) g; (void) rows; return 0; }
-
 int32_t launch_recurrence(const RecurArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
     SK_REQUIRE(a.g.kdim <= RECUR_MAX_KDIM, "recurrence: key size %d (at most %d)", a.g.kdim, RECUR_MAX_KDIM);
+    if (a.map.seq >= 0 && !a.f32_act && a.work && a.rows >= RECUR_CHUNK_MIN_ROWS && recur_work_bytes(a.g, a.rows) > 0) return launch_recur_chunks(a, s);
     SK_TRY(a.g.delta ? run_step_rows<true>(a, s) : run_step_rows<false>(a, s));
     if (a.map.seq >= 0) SK_CUDA(launch_pdl(recur_tail_kernel, dim3((a.g.conv_dim() + 255) / 256, std::min(a.rows, a.g.taps)), dim3(256), 0, s, a));
     return SKAINET_CUDA_OK;

@@ -49,8 +49,12 @@ struct RecurArgs {
 // A sequence at position 0 starts from a zero state and zero inputs whatever its store holds.
 int32_t launch_recurrence(const RecurArgs& a, cudaStream_t s);
 
-// Bytes of RecurArgs::work for passes of up to `rows` tokens.
+// Bytes of RecurArgs::work for passes of up to `rows` tokens; 0 when the tile kernels do not take the geometry.
 size_t recur_work_bytes(const RecurGeom& g, int rows);
+
+// recurrence_chunk.cu: `rows` tokens of one sequence
+constexpr int RECUR_CHUNK_MIN_ROWS = 12;
+int32_t launch_recur_chunks(const RecurArgs& a, cudaStream_t s);
 
 // y = o normed in parts of `part` columns, times gain, gated by silu(z), in the activation type.
 //   gate_first: norm(o * silu(z)) * gain[column];  else norm(o) * gain[column % part] * silu(z)
@@ -69,3 +73,18 @@ struct GatedNormArgs {
 int32_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s);
 
 }  // namespace sk
+
+#ifdef __CUDACC__
+namespace skd {
+
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+
+// Input of convolution channel c at position p; rows of the pass start at position pos0 in row row0.
+__device__ __forceinline__ float conv_input(const sk::RecurArgs& a, const float* tail, int row0, int pos0, int p, int c) {
+    if (p < 0) return 0.0f;
+    if (p >= pos0) return a.proj[(size_t) (row0 + p - pos0) * a.proj_ld + a.conv_off + c];
+    return tail[(size_t) (p % a.g.taps) * a.g.conv_dim() + c];
+}
+
+}  // namespace skd
+#endif
