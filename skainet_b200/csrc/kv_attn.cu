@@ -2,7 +2,7 @@
 //
 //   kv_prep_kernel       biases, unit-rms queries and keys, ring append.
 //   kv_attn_tile_kernel  bf16: the MMA rows are (activation row, head) pairs that share a key/value head, so a staged key or value
-//                        row serves the whole group. In prompts each of eight warps owns 16 pairs and all read the same tile of 64
+//                        row serves the whole group. In prompts each of four warps owns 16 pairs and all read the same tile of 64
 //                        keys; in a decode step four warps own the same 16 pairs and a quarter of the tile's keys each. Keys may
 //                        be split over CTAs; kv_merge_kernel joins the parts in fixed order.
 //   kv_attn_rows_kernel  fp32 FMA, one CTA per (row, head), any size: the 32-bit mode, and bf16 models whose heads are too large
@@ -107,15 +107,17 @@ __global__ void __launch_bounds__(RK) kv_attn_rows_kernel(const KvAttnArgs a) {
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int TK = 64;                       // keys of a staged tile
 
+__device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+
 // Widths up to 16 * KS (keys) and 8 * VN (values). DECODE: the activation rows of a CTA are one, its warps split the keys.
 template <int KS, int VN, bool DECODE>
 struct TileShape {
-    static constexpr int WARPS = DECODE ? 4 : 8, ROWS = DECODE ? 16 : 128, KEYS = DECODE ? TK / WARPS : TK;   // pairs of a CTA, keys of a warp
+    static constexpr int WARPS = 4, ROWS = DECODE ? 16 : 64, KEYS = DECODE ? TK / WARPS : TK;   // pairs of a CTA, keys of a warp
     static constexpr int STAGES = DECODE ? 3 : 2;
-    static constexpr bool Q_REGS = KS <= 8;
+    static constexpr bool Q_REGS = KS <= 8;                      // queries live in registers and pass through the last stage's key tile
     // rows are 16 bytes longer than the data: an odd number of 16-byte units, so ldmatrix rows meet different banks
     static __host__ __device__ int smem(int kld, int vcld) {
-        const int tiles = (ROWS * (kld + 8) + STAGES * TK * (kld + 8 + vcld + 8)) * 2, merge = DECODE ? WARPS * 16 * (vcld + 2) * 4 : 0;
+        const int tiles = ((Q_REGS ? 0 : ROWS * (kld + 8)) + STAGES * TK * (kld + 8 + vcld + 8)) * 2, merge = DECODE ? WARPS * 16 * (vcld + 2) * 4 : 0;
         return tiles > merge ? tiles : merge;
     }
 };
@@ -133,7 +135,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     const int tiles_m = DECODE ? (group + 15) / 16 : 0;
     const int m_tile = DECODE ? (int) blockIdx.x % tiles_m : (int) (gridDim.x - 1 - blockIdx.x);          // the longest prompt tiles first
     const int row_base = DECODE ? (int) blockIdx.x / tiles_m : 0, p0 = m_tile * S::ROWS, pairs = DECODE ? group : a.rows * group;
-    const uint32_t sq = skd::smem_u32(raw), sk = sq + S::ROWS * klds * 2, sv = sk + S::STAGES * TK * klds * 2;
+    const uint32_t sk = skd::smem_u32(raw), sv = sk + S::STAGES * TK * klds * 2, sq = S::Q_REGS ? sk + (S::STAGES - 1) * TK * klds * 2 : sv + S::STAGES * TK * vlds * 2;
     skd::pdl_launch_dependents();
     skd::pdl_wait();
     const int seq = a.map.seq_of(row_base);
@@ -146,14 +148,16 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     if (splits > 1) { const int per = (t1 + splits - 1) / splits; t0 = min(t1, split * per); t1 = min(t1, t0 + per); }
 
     auto load_tile = [&](int t, int stage) {
-        const int j0 = lo + t * TK, kch = kld / 8, vch = vcld / 8, slot0 = j0 % a.cache.cap;
-        for (int i = threadIdx.x; i < TK * (kch + vch); i += S::WARPS * 32) {
-            const bool is_v = i >= TK * kch;
-            const int e = is_v ? i - TK * kch : i, ch = is_v ? vch : kch, r = e / ch, c = e % ch;
-            int slot = slot0 + r;
+        const int kch = kld / 8, both = kch + vcld / 8;
+        int slot = (lo + t * TK + warp) % a.cache.cap;              // a warp copies a key and its value
+#pragma unroll 4
+        for (int r = warp; r < TK; r += S::WARPS) {
+            for (int c = lane; c < both; c += 32) {
+                if (c < kch) skd::cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
+                else skd::cp16(sv + ((stage * TK + r) * vlds + (c - kch) * 8) * 2, vc + (size_t) slot * vcld + (c - kch) * 8);
+            }
+            slot += S::WARPS;
             if (slot >= a.cache.cap) slot %= a.cache.cap;
-            if (is_v) skd::cp16(sv + ((stage * TK + r) * vlds + c * 8) * 2, vc + (size_t) slot * vcld + c * 8);
-            else skd::cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
         }
     };
     // queries; rows past the last pair repeat it and are not stored
@@ -161,6 +165,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
         const int r = i / (kld / 8), c = i % (kld / 8), p = min(p0 + r, pairs - 1);
         skd::cp16(sq + (r * klds + c * 8) * 2, (const bf16*) a.q + ((size_t) (row_base + p / group) * g.heads + kh * group + p % group) * kld + c * 8);
     }
+    skd::cp_commit();
 #pragma unroll
     for (int s = 0; s < S::STAGES - 1; ++s) { if (t0 + s < t1) load_tile(t0 + s, s); skd::cp_commit(); }
 
@@ -183,6 +188,12 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     const uint32_t k_at = sk + ((k0w + (lane & 7) + (lane >> 4) * 8) * klds + ((lane >> 3) & 1) * 8) * 2;
     const uint32_t v_at = sv + ((k0w + (lane & 7) + ((lane >> 3) & 1) * 8) * vlds + (lane >> 4) * 8) * 2;
     const float sc2 = a.scale * LOG2E;
+    if (S::Q_REGS) {
+        skd::cp_wait<S::STAGES - 1>();
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < KS; ++k) if (k < ks_n) skd::ldsm4(qf[S::Q_REGS ? k : 0], q_at + k * 32);
+    }
     constexpr int NK = S::KEYS / 8;
 
     for (int t = t0; t < t1; ++t) {
@@ -191,9 +202,6 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
         __syncthreads();
         if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES);
         skd::cp_commit();
-        if (S::Q_REGS && t == t0)
-#pragma unroll
-            for (int k = 0; k < KS; ++k) if (k < ks_n) skd::ldsm4(qf[S::Q_REGS ? k : 0], q_at + k * 32);
         float c[NK][4];
 #pragma unroll
         for (int n = 0; n < NK; ++n)
@@ -216,18 +224,22 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
         const int j0 = lo + t * TK + k0w;
         const bool whole = j0 >= lo_last && j0 + S::KEYS - 1 <= pos_first;
         float mx[2] = {m[0], m[1]};
+        if (!whole)
+#pragma unroll
+            for (int n = 0; n < NK; ++n)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int j = j0 + n * 8 + tq * 2 + (i & 1);
+                    if (j < lo_r[i >> 1] || j > pos_r[i >> 1]) c[n][i] = -INFINITY;
+                }
 #pragma unroll
         for (int n = 0; n < NK; ++n)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int j = j0 + n * 8 + tq * 2 + (i & 1);
-                c[n][i] = whole || (j >= lo_r[i >> 1] && j <= pos_r[i >> 1]) ? c[n][i] * sc2 : -INFINITY;
-                mx[i >> 1] = fmaxf(mx[i >> 1], c[n][i]);
-            }
+            for (int i = 0; i < 4; ++i) { c[n][i] *= sc2; mx[i >> 1] = fmaxf(mx[i >> 1], c[n][i]); }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             mx[i] = fmaxf(mx[i], __shfl_xor_sync(~0u, mx[i], 1)); mx[i] = fmaxf(mx[i], __shfl_xor_sync(~0u, mx[i], 2));
-            const float fade = exp2f(m[i] - mx[i]);
+            const float fade = ex2(m[i] - mx[i]);
             m[i] = mx[i];
             l[i] *= fade;
             if (__any_sync(~0u, fade != 1.0f))
@@ -237,7 +249,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
 #pragma unroll
         for (int n = 0; n < NK; ++n)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) { c[n][i] = exp2f(c[n][i] - m[i >> 1]); l[i >> 1] += c[n][i]; }
+            for (int i = 0; i < 4; ++i) { c[n][i] = ex2(c[n][i] - m[i >> 1]); l[i >> 1] += c[n][i]; }
 #pragma unroll
         for (int k = 0; k < NK / 2; ++k) {
             const uint32_t p[4] = {skd::pack_bf16(c[2 * k][0], c[2 * k][1]), skd::pack_bf16(c[2 * k][2], c[2 * k][3]), skd::pack_bf16(c[2 * k + 1][0], c[2 * k + 1][1]),
@@ -328,13 +340,28 @@ __global__ void __launch_bounds__(128) kv_merge_kernel(const KvAttnArgs a, int s
     for (int s = lane; s < splits; s += 32) top = fmaxf(top, rec[(size_t) s * ld + g.vcld()]);
     top = skd::warp_max(top);
     float den = 0.0f;
-    if (a.sink) { const float s2 = a.sink[h] * LOG2E; top = fmaxf(top, s2); den = exp2f(s2 - top); }
-    for (int s = 0; s < splits; ++s) den += rec[(size_t) s * ld + g.vcld() + 1] * exp2f(rec[(size_t) s * ld + g.vcld()] - top);
-    for (int d = lane; d < g.vdim; d += 32) {
-        float v = 0.0f;
-#pragma unroll 4
-        for (int s = 0; s < splits; ++s) v = fmaf(rec[(size_t) s * ld + d], exp2f(rec[(size_t) s * ld + g.vcld()] - top), v);
-        ((bf16*) a.out)[(size_t) row * g.out_ld() + h * g.vdim + d] = __float2bfloat16_rn(v / den);
+    if (a.sink) { const float s2 = a.sink[h] * LOG2E; top = fmaxf(top, s2); if (lane == 0) den = exp2f(s2 - top); }
+    for (int s = lane; s < splits; s += 32) den += rec[(size_t) s * ld + g.vcld() + 1] * exp2f(rec[(size_t) s * ld + g.vcld()] - top);
+    den = skd::warp_sum(den);
+    // lanes own pairs of columns; the factors of 32 splits at a time come from the lanes that computed them
+    for (int d0 = 0; d0 < g.vcld(); d0 += 64) {
+        const int d = d0 + 2 * lane;
+        const bool live = d < g.vcld();
+        float2 v = make_float2(0.0f, 0.0f);
+        for (int s0 = 0; s0 < splits; s0 += 32) {
+            const float f = s0 + lane < splits ? exp2f(rec[(size_t) (s0 + lane) * ld + g.vcld()] - top) : 0.0f;
+#pragma unroll 8
+            for (int i = 0; i < 32; ++i) {
+                const float fi = __shfl_sync(~0u, f, i);
+                if (s0 + i >= splits) break;
+                if (!live) continue;
+                const float2 x = *reinterpret_cast<const float2*>(rec + (size_t) (s0 + i) * ld + d);
+                v.x = fmaf(x.x, fi, v.x); v.y = fmaf(x.y, fi, v.y);
+            }
+        }
+        bf16* out = (bf16*) a.out + (size_t) row * g.out_ld() + h * g.vdim;
+        if (d < g.vdim) out[d] = __float2bfloat16_rn(v.x / den);
+        if (d + 1 < g.vdim) out[d + 1] = __float2bfloat16_rn(v.y / den);
     }
 }
 

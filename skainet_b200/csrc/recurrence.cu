@@ -4,7 +4,6 @@
 //                        registers (columns of the state never meet), so a step reads and writes the state once.
 //   recur_tail_kernel    the convolution inputs a prompt pass leaves for the next one.
 //   recurrence_chunk.cu  prompts of bf16 models: chunks of 64 tokens on the tensor cores.
-//   gated_norm_kernel    norm and output gate.
 #include "recurrence.cuh"
 #include "tma.cuh"
 
@@ -152,43 +151,6 @@ int32_t run_step_rows(const RecurArgs& a, cudaStream_t s) {
     return run_step<DELTA, 16>(a, s);
 }
 
-// GROUP threads share a part: 32 (several parts per CTA) or 256.
-template <typename T, int GROUP>
-__global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormArgs a) {
-    __shared__ float sh[8];
-    skd::pdl_launch_dependents();
-    skd::pdl_wait();
-    const int parts = a.cols / a.part, tid = threadIdx.x % GROUP;
-    const int64_t unit = (int64_t) blockIdx.x * (256 / GROUP) + threadIdx.x / GROUP;
-    if (GROUP == 32 && unit >= (int64_t) a.rows * parts) return;
-    const int row = (int) (unit / parts), c0 = (int) (unit % parts) * a.part;
-    const float *o = a.o + (size_t) row * a.cols + c0, *z = a.z + (size_t) row * a.z_ld + c0;
-    T* y = (T*) a.act + (size_t) row * a.act_ld + c0;
-    const float* gain = a.gate_first ? a.gain + c0 : a.gain;
-    float ss = 0.0f;
-    for (int c = tid; c < a.part; c += GROUP) {
-        const float v = a.gate_first ? o[c] * skd::silu(z[c]) : o[c];
-        ss = fmaf(v, v, ss);
-    }
-    ss = skd::warp_sum(ss);
-    if (GROUP > 32) {
-        if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = ss;
-        __syncthreads();
-        ss = 0.0f;
-        for (int i = 0; i < GROUP / 32; ++i) ss += sh[i];
-    }
-    const float r = 1.0f / sqrtf(ss / (float) a.part + a.eps);
-    for (int c = tid; c < a.part; c += GROUP) skd::store_act(y + c, o[c] * skd::silu(z[c]) * r * gain[c]);
-}
-
-template <typename T>
-int32_t run_gated_norm(const GatedNormArgs& a, cudaStream_t s) {
-    const int64_t units = (int64_t) a.rows * (a.cols / a.part);
-    if (a.part <= 512) SK_CUDA(launch_pdl(gated_norm_kernel<T, 32>, dim3((unsigned) ((units + 7) / 8)), dim3(256), 0, s, a));
-    else SK_CUDA(launch_pdl(gated_norm_kernel<T, 256>, dim3((unsigned) units), dim3(256), 0, s, a));
-    return SKAINET_CUDA_OK;
-}
-
 }  // namespace
 
 int32_t launch_recurrence(const RecurArgs& a, cudaStream_t s) {
@@ -198,11 +160,6 @@ int32_t launch_recurrence(const RecurArgs& a, cudaStream_t s) {
     SK_TRY(a.g.delta ? run_step_rows<true>(a, s) : run_step_rows<false>(a, s));
     if (a.map.seq >= 0) SK_CUDA(launch_pdl(recur_tail_kernel, dim3((a.g.conv_dim() + 255) / 256, std::min(a.rows, a.g.taps)), dim3(256), 0, s, a));
     return SKAINET_CUDA_OK;
-}
-
-int32_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s) {
-    if (a.rows <= 0) return SKAINET_CUDA_OK;
-    return a.f32_act ? run_gated_norm<float>(a, s) : run_gated_norm<bf16>(a, s);
 }
 
 }  // namespace sk

@@ -56,22 +56,6 @@ size_t recur_work_bytes(const RecurGeom& g, int rows);
 constexpr int RECUR_CHUNK_MIN_ROWS = 12;
 int32_t launch_recur_chunks(const RecurArgs& a, cudaStream_t s);
 
-// y = o normed in parts of `part` columns, times gain, gated by silu(z), in the activation type.
-//   gate_first: norm(o * silu(z)) * gain[column];  else norm(o) * gain[column % part] * silu(z)
-struct GatedNormArgs {
-    const float* o = nullptr;              // [row][cols]
-    const float* z = nullptr;              // [row][z_ld]
-    int z_ld = 0;
-    const float* gain = nullptr;
-    bool gate_first = false;
-    int part = 0, cols = 0, rows = 0;
-    float eps = 0.0f;
-    void* act = nullptr;
-    int act_ld = 0;
-    bool f32_act = false;
-};
-int32_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s);
-
 }  // namespace sk
 
 #ifdef __CUDACC__

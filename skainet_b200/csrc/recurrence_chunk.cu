@@ -108,6 +108,79 @@ __global__ void __launch_bounds__(256) recur_conv_kernel(const RecurArgs a, cons
     }
 }
 
+// The same for four taps and sizes that fill the tiles: a warp owns 128 channels (four per lane) of 16 rows and slides over them
+// in registers. grid: (16 rows, groups of eight warps over q and k vectors | v channels | 32 heads' step sizes)
+__global__ void __launch_bounds__(256) recur_conv4_kernel(const RecurArgs a, const Work w, int v_blocks) {
+    const RecurGeom& g = a.g;
+    const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, row0 = blockIdx.x * CONV_ROWS, qk_units = 2 * g.groups;
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    if (unit >= qk_units + v_blocks) {
+        const int h = (unit - qk_units - v_blocks) * 32 + lane;
+        if (h >= g.heads) return;
+        const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h];
+#pragma unroll 4
+        for (int r = 0; r < CONV_ROWS; ++r) {
+            const int row = row0 + r;
+            float ld = 0.0f, st = 0.0f;
+            if (row < a.rows) {
+                const float* p = a.proj + (size_t) row * a.proj_ld;
+                const float dt = skd::softplus(p[a.dt_off + h] + bias);
+                ld = neg_a * dt;
+                st = g.delta ? skd::sigmoid(p[a.beta_off + h]) : dt;
+            }
+            w.log_decay[(size_t) h * w.rows + row] = ld; w.step[(size_t) h * w.rows + row] = st;
+        }
+        return;
+    }
+    const bool is_v = unit >= qk_units;
+    const int u = unit;                                             // q or k vector
+    int ch, out_ld;
+    bf16* out;
+    bool live;
+    if (is_v) {
+        const int c = (unit - qk_units) * 128 + 4 * lane, h = c / g.vdim;
+        live = c < g.v_dim();
+        ch = a.v_off + c; out_ld = w.vp;
+        out = w.v + (size_t) h * w.rows * w.vp + c % g.vdim;
+    } else {
+        live = 4 * lane < g.kdim;
+        ch = (u < g.groups ? a.q_off + u * g.kdim : a.k_off + (u - g.groups) * g.kdim) + 4 * lane; out_ld = w.kp;
+        out = w.qk + (size_t) u * w.rows * w.kp + 4 * lane;
+    }
+    const int pos0 = a.map.pos[a.map.seq];
+    const float* tail = a.tail + (size_t) a.map.seq * g.tail_size();
+    auto input = [&](int row) {
+        if (!live || pos0 + row < 0 || row >= a.rows) return make_float4(0, 0, 0, 0);
+        const float* p = row >= 0 ? a.proj + (size_t) row * a.proj_ld + a.conv_off + ch : tail + (size_t) ((pos0 + row) % 4) * g.conv_dim() + ch;
+        return *reinterpret_cast<const float4*>(p);
+    };
+    float4 wt[4], bias = make_float4(0, 0, 0, 0);                   // taps of channel ch + i
+#pragma unroll
+    for (int i = 0; i < 4; ++i) wt[i] = live ? *reinterpret_cast<const float4*>(a.conv_w + (size_t) (ch + i) * 4) : make_float4(0, 0, 0, 0);
+    if (live && a.conv_b) bias = make_float4(a.conv_b[ch], a.conv_b[ch + 1], a.conv_b[ch + 2], a.conv_b[ch + 3]);
+    float4 x0 = input(row0 - 3), x1 = input(row0 - 2), x2 = input(row0 - 1);
+#pragma unroll 8
+    for (int r = 0; r < CONV_ROWS; ++r) {
+        const int row = row0 + r;
+        const float4 x3 = input(row);
+        float4 y;
+        y.x = skd::silu(fmaf(wt[0].w, x3.x, fmaf(wt[0].z, x2.x, fmaf(wt[0].y, x1.x, fmaf(wt[0].x, x0.x, bias.x)))));
+        y.y = skd::silu(fmaf(wt[1].w, x3.y, fmaf(wt[1].z, x2.y, fmaf(wt[1].y, x1.y, fmaf(wt[1].x, x0.y, bias.y)))));
+        y.z = skd::silu(fmaf(wt[2].w, x3.z, fmaf(wt[2].z, x2.z, fmaf(wt[2].y, x1.z, fmaf(wt[2].x, x0.z, bias.z)))));
+        y.w = skd::silu(fmaf(wt[3].w, x3.w, fmaf(wt[3].z, x2.w, fmaf(wt[3].y, x1.w, fmaf(wt[3].x, x0.w, bias.w)))));
+        x0 = x1; x1 = x2; x2 = x3;
+        uint2 b = make_uint2(skd::pack_bf16(y.x, y.y), skd::pack_bf16(y.z, y.w));
+        if (row >= a.rows) b = make_uint2(0, 0);
+        if (live) *reinterpret_cast<uint2*>(out + (size_t) row * out_ld) = b;
+        if (!is_v) {
+            const float e0 = skd::bf16_lo(b.x), e1 = skd::bf16_hi(b.x), e2 = skd::bf16_lo(b.y), e3 = skd::bf16_hi(b.y);
+            const float ss = skd::warp_sum(live ? fmaf(e0, e0, fmaf(e1, e1, fmaf(e2, e2, e3 * e3))) : 0.0f);
+            if (lane == 0) w.length[(size_t) u * w.rows + row] = row >= a.rows ? 0.0f : g.delta ? 1.0f / sqrtf(ss + 1e-6f) * (u < g.groups ? a.q_scale : 1.0f) : 1.0f;
+        }
+    }
+}
+
 // Sums of the log decays up to every token of a chunk; lane l holds tokens 2l and 2l + 1.
 __device__ __forceinline__ void decay_sums(float a, float b, int lane, double (&g)[2]) {
     double s = (double) a + (double) b;
@@ -513,9 +586,15 @@ size_t recur_work_bytes(const RecurGeom& g, int rows) {
 int32_t launch_recur_chunks(const RecurArgs& a, cudaStream_t s) {
     const RecurGeom& g = a.g;
     const Work w = layout(g, a.rows, a.work);
-    const int conv_bytes = (CONV_ROWS + g.taps - 1) * std::max(g.kdim, g.vdim) * (int) sizeof(float);
-    SK_TRY(ensure_dynamic_smem((const void*) recur_conv_kernel, conv_bytes));
-    SK_CUDA(launch_pdl(recur_conv_kernel, dim3(w.rows / CONV_ROWS, 2 * g.groups + g.heads), dim3(256), conv_bytes, s, a, w));
+    const bool quads = (a.proj_ld | a.conv_off | a.q_off | a.k_off | a.v_off) % 4 == 0;
+    if (g.taps == 4 && quads && g.kdim == w.kp && g.kdim <= 128 && g.vdim == w.vp) {
+        const int v_blocks = (g.v_dim() + 127) / 128, units = 2 * g.groups + v_blocks + (g.heads + 31) / 32;
+        SK_CUDA(launch_pdl(recur_conv4_kernel, dim3(w.rows / CONV_ROWS, (units + 7) / 8), dim3(256), 0, s, a, w, v_blocks));
+    } else {
+        const int conv_bytes = (CONV_ROWS + g.taps - 1) * std::max(g.kdim, g.vdim) * (int) sizeof(float);
+        SK_TRY(ensure_dynamic_smem((const void*) recur_conv_kernel, conv_bytes));
+        SK_CUDA(launch_pdl(recur_conv_kernel, dim3(w.rows / CONV_ROWS, 2 * g.groups + g.heads), dim3(256), conv_bytes, s, a, w));
+    }
     if (!g.delta) {
         if (state_cols(g) == 64) return w.kp <= 128 ? run_scan<false, 64, 2>(a, w, s) : run_scan<false, 64, 4>(a, w, s);
         return w.kp <= 128 ? run_scan<false, 32, 2>(a, w, s) : run_scan<false, 32, 4>(a, w, s);

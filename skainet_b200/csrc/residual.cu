@@ -208,6 +208,81 @@ __global__ void __launch_bounds__(RT) embed_pos_kernel(const EmbedPosArgs a) {
     if (cs > 1) cl.sync();
 }
 
+// A part of up to 512 columns per warp, its values in registers.
+constexpr int GN_COLS = 512;
+template <typename T, int V>
+__global__ void __launch_bounds__(RT) gated_norm_warp_kernel(const GatedNormArgs a) {
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    const int parts = a.cols / a.part, lane = threadIdx.x & 31;
+    const int64_t unit = (int64_t) blockIdx.x * (RT / 32) + (threadIdx.x >> 5);
+    if (unit >= (int64_t) a.rows * parts) return;
+    const int row = (int) (unit / parts), c0 = (int) (unit % parts) * a.part;
+    const float *o = a.o + (size_t) row * a.cols + c0, *z = a.z + (size_t) row * a.z_ld + c0, *gain = a.gate_first ? a.gain + c0 : a.gain;
+    Vec<V> v[GN_COLS / 32 / V];
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < GN_COLS / 32 / V; ++k) {
+        const int c = (k * 32 + lane) * V;
+        if (c >= a.part) break;
+        v[k] = ld<V>(o + c);
+        const Vec<V> g = ld<V>(z + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            const float y = v[k].v[i] * skd::silu(g.v[i]);
+            const float n = a.gate_first ? y : v[k].v[i];
+            ss = fmaf(n, n, ss);
+            v[k].v[i] = y;
+        }
+    }
+    const float r = 1.0f / sqrtf(skd::warp_sum(ss) / (float) a.part + a.eps);
+#pragma unroll
+    for (int k = 0; k < GN_COLS / 32 / V; ++k) {
+        const int c = (k * 32 + lane) * V;
+        if (c >= a.part) break;
+        const Vec<V> g = ld<V>(gain + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[k].v[i] *= r * g.v[i];
+        st_act<V>((T*) a.act + (size_t) row * a.act_ld + c0 + c, v[k]);
+    }
+}
+// A wider part per cluster.
+template <typename T, int V>
+__global__ void __launch_bounds__(RT) gated_norm_kernel(const GatedNormArgs a) {
+    namespace cg = cooperative_groups;
+    extern __shared__ __align__(16) float sx[];
+    __shared__ float sh[RT / 32], part;
+    skd::pdl_launch_dependents();
+    skd::pdl_wait();
+    cg::cluster_group cl = cg::this_cluster();
+    const int cs = (int) cl.num_blocks(), rank = (int) cl.block_rank(), unit = blockIdx.x / cs, parts = a.cols / a.part, row = unit / parts, c0 = unit % parts * a.part;
+    const Span sp = cluster_span(a.part, cs, rank);
+    const float *o = a.o + (size_t) row * a.cols + c0, *z = a.z + (size_t) row * a.z_ld + c0, *gain = a.gate_first ? a.gain + c0 : a.gain;
+    float ss = 0.0f;
+#pragma unroll 4
+    for (int c = sp.c0 + (int) threadIdx.x * V; c < sp.c1; c += RT * V) {
+        Vec<V> v = ld<V>(o + c);
+        const Vec<V> g = ld<V>(z + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            const float y = v.v[i] * skd::silu(g.v[i]);
+            const float n = a.gate_first ? y : v.v[i];
+            ss = fmaf(n, n, ss);
+            v.v[i] = y;
+        }
+        st<V>(sx + c - sp.c0, v);
+    }
+    const float r = 1.0f / sqrtf(cluster_sum(ss, sh, &part, cl, cs) / (float) a.part + a.eps);
+    for (int c = sp.c0 + (int) threadIdx.x * V; c < sp.c1; c += RT * V) {
+        Vec<V> v = ld<V>(sx + c - sp.c0);
+        const Vec<V> g = ld<V>(gain + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v.v[i] *= r * g.v[i];
+        st_act<V>((T*) a.act + (size_t) row * a.act_ld + c0 + c, v);
+    }
+    if (cs > 1) cl.sync();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(RT) embed_rows_kernel(const bf16* __restrict__ table, int ld_, const int32_t* __restrict__ ids, int cols, int vocab,
                                                         float* __restrict__ x, float* __restrict__ state0, T* __restrict__ act, int act_ld) {
@@ -235,15 +310,15 @@ __global__ void __launch_bounds__(RT) row_norm_kernel(const float* __restrict__ 
     for (int c = threadIdx.x; c < cols; c += RT) skd::store_act(act + (size_t) blockIdx.x * act_ld + c, gains ? p[c] * r * gains[c] : p[c] * r);
 }
 
-// One cluster per row; a CTA keeps its columns of the row in dynamic shared memory.
+// One cluster per row (of `cols` columns, `rows` of them); a CTA keeps its columns of the row in dynamic shared memory.
 template <typename A>
-int32_t run_row_clusters(void (*kernel)(const A), const A& a, cudaStream_t s) {
+int32_t run_row_clusters(void (*kernel)(const A), const A& a, int rows, int cols, cudaStream_t s) {
     int cs = 1;                                                 // CTAs per row: while the machine has room and a CTA keeps 256 columns
-    while (cs < 8 && a.rows * cs * 2 <= sm_count() && a.cols / (cs * 2) >= 256) cs *= 2;
-    const int per = ((a.cols + cs - 1) / cs + 3) / 4 * 4;
+    while (cs < 8 && rows * cs * 2 <= sm_count() && cols / (cs * 2) >= 256) cs *= 2;
+    const int per = ((cols + cs - 1) / cs + 3) / 4 * 4;
     SK_TRY(ensure_dynamic_smem((const void*) kernel, per * (int) sizeof(float)));
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(a.rows * cs); cfg.blockDim = dim3(RT); cfg.dynamicSmemBytes = per * sizeof(float); cfg.stream = s;
+    cfg.gridDim = dim3(rows * cs); cfg.blockDim = dim3(RT); cfg.dynamicSmemBytes = per * sizeof(float); cfg.stream = s;
     cudaLaunchAttribute at[2];
     at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = 1;
     at[1].id = cudaLaunchAttributeClusterDimension; at[1].val.clusterDim.x = cs; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
@@ -252,25 +327,40 @@ int32_t run_row_clusters(void (*kernel)(const A), const A& a, cudaStream_t s) {
     return SKAINET_CUDA_OK;
 }
 
+template <typename T>
+int32_t run_gated_norm(const GatedNormArgs& a, cudaStream_t s) {
+    const int64_t units = (int64_t) a.rows * (a.cols / a.part);
+    SK_REQUIRE(units < (1 << 28), "gated_norm: too many parts");
+    const bool vec = a.part % 4 == 0 && a.z_ld % 4 == 0 && ((uintptr_t) a.z & 15) == 0;
+    if (a.part > GN_COLS) return run_row_clusters(vec ? gated_norm_kernel<T, 4> : gated_norm_kernel<T, 1>, a, (int) units, a.part, s);
+    SK_CUDA(launch_pdl(vec ? gated_norm_warp_kernel<T, 4> : gated_norm_warp_kernel<T, 1>, dim3((unsigned) ((units + RT / 32 - 1) / (RT / 32))), dim3(RT), 0, s, a));
+    return SKAINET_CUDA_OK;
+}
+
 }  // namespace
 
 int32_t launch_sublayer(const SublayerArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
     const bool vec = a.cols % 4 == 0 && a.act_ld % 4 == 0 && a.state_stride % 4 == 0;
-    if (a.f32_act) return run_row_clusters(vec ? sublayer_kernel<float, 4> : sublayer_kernel<float, 1>, a, s);
-    return run_row_clusters(vec ? sublayer_kernel<bf16, 4> : sublayer_kernel<bf16, 1>, a, s);
+    if (a.f32_act) return run_row_clusters(vec ? sublayer_kernel<float, 4> : sublayer_kernel<float, 1>, a, a.rows, a.cols, s);
+    return run_row_clusters(vec ? sublayer_kernel<bf16, 4> : sublayer_kernel<bf16, 1>, a, a.rows, a.cols, s);
 }
 
 int32_t launch_sandwich(const SandwichArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
     const bool vec = a.cols % 4 == 0 && a.act_ld % 4 == 0;
-    if (a.f32_act) return run_row_clusters(vec ? sandwich_kernel<float, 4> : sandwich_kernel<float, 1>, a, s);
-    return run_row_clusters(vec ? sandwich_kernel<bf16, 4> : sandwich_kernel<bf16, 1>, a, s);
+    if (a.f32_act) return run_row_clusters(vec ? sandwich_kernel<float, 4> : sandwich_kernel<float, 1>, a, a.rows, a.cols, s);
+    return run_row_clusters(vec ? sandwich_kernel<bf16, 4> : sandwich_kernel<bf16, 1>, a, a.rows, a.cols, s);
 }
 
 int32_t launch_embed_pos(const EmbedPosArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
-    return a.f32_act ? run_row_clusters(embed_pos_kernel<float>, a, s) : run_row_clusters(embed_pos_kernel<bf16>, a, s);
+    return a.f32_act ? run_row_clusters(embed_pos_kernel<float>, a, a.rows, a.cols, s) : run_row_clusters(embed_pos_kernel<bf16>, a, a.rows, a.cols, s);
+}
+
+int32_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return SKAINET_CUDA_OK;
+    return a.f32_act ? run_gated_norm<float>(a, s) : run_gated_norm<bf16>(a, s);
 }
 
 int32_t launch_embed_rows(const bf16* table, int ld_, const int32_t* ids, int rows, int cols, int vocab, float* x, float* state0, void* act, int act_ld,

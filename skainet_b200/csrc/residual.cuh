@@ -1,5 +1,5 @@
 // What stands between the sublayers: residual sum and RMS norms of the sublayer outputs (one number, or one per coordinate),
-// of the next sublayer's input, and the depth average over the earlier layers' results. Everything here is fp32; only the copy
+// of the next sublayer's input, of a mixer's gated output, and the depth average over the earlier layers' results. Everything here is fp32; only the copy
 // the next linear reads is narrowed.
 #pragma once
 #include "linear_bf16.cuh"
@@ -61,6 +61,22 @@ struct EmbedPosArgs {
     bool f32_act = false;
 };
 int32_t launch_embed_pos(const EmbedPosArgs& a, cudaStream_t s);
+
+// y = o normed in parts of `part` columns, times gain, gated by silu(z), in the activation type.
+//   gate_first: norm(o * silu(z)) * gain[column];  else norm(o) * gain[column % part] * silu(z)
+struct GatedNormArgs {
+    const float* o = nullptr;              // [row][cols]
+    const float* z = nullptr;              // [row][z_ld]
+    int z_ld = 0;
+    const float* gain = nullptr;
+    bool gate_first = false;
+    int part = 0, cols = 0, rows = 0;
+    float eps = 0.0f;
+    void* act = nullptr;
+    int act_ld = 0;
+    bool f32_act = false;
+};
+int32_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s);
 
 // act[i] = rmsnorm(x[index ? index[i] : i]) * gain[c] for i < rows
 int32_t launch_row_norm(const float* x, const int32_t* index, int rows, int cols, const float* gain, float eps, void* act, int act_ld, bool f32_act, cudaStream_t s);
