@@ -328,41 +328,41 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     }
 }
 
-// One warp per (row, head): the records of the splits, then the sink.
+// One CTA per (row, head): its four warps take a quarter of the splits each; then the sink.
 __global__ void __launch_bounds__(128) kv_merge_kernel(const KvAttnArgs a, int splits) {
+    extern __shared__ float dyn[];                                // factors [splits] | sums [4][vcld]
     skd::pdl_launch_dependents();
     skd::pdl_wait();
     const KvGeom& g = a.g;
-    const int h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, row = blockIdx.x, ld = g.vcld() + 2;
-    if (h >= g.heads) return;
+    const int row = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, vcld = g.vcld(), ld = vcld + 2;
     const float* rec = a.part + ((size_t) row * g.heads + h) * splits * ld;
-    float top = NEG_BIG;
-    for (int s = lane; s < splits; s += 32) top = fmaxf(top, rec[(size_t) s * ld + g.vcld()]);
+    float *f = dyn, *sum = dyn + splits;
+    // every warp forms the joint maximum and denominator; warp 0 leaves the factors
+    float top = a.sink ? a.sink[h] * LOG2E : NEG_BIG, den = 0.0f;
+    if (a.sink && lane == 0) den = 1.0f;
+    const float s2 = top;
+    for (int s = lane; s < splits; s += 32) top = fmaxf(top, rec[(size_t) s * ld + vcld]);
     top = skd::warp_max(top);
-    float den = 0.0f;
-    if (a.sink) { const float s2 = a.sink[h] * LOG2E; top = fmaxf(top, s2); if (lane == 0) den = exp2f(s2 - top); }
-    for (int s = lane; s < splits; s += 32) den += rec[(size_t) s * ld + g.vcld() + 1] * exp2f(rec[(size_t) s * ld + g.vcld()] - top);
-    den = skd::warp_sum(den);
-    // lanes own pairs of columns; the factors of 32 splits at a time come from the lanes that computed them
-    for (int d0 = 0; d0 < g.vcld(); d0 += 64) {
-        const int d = d0 + 2 * lane;
-        const bool live = d < g.vcld();
-        float2 v = make_float2(0.0f, 0.0f);
-        for (int s0 = 0; s0 < splits; s0 += 32) {
-            const float f = s0 + lane < splits ? exp2f(rec[(size_t) (s0 + lane) * ld + g.vcld()] - top) : 0.0f;
-#pragma unroll 8
-            for (int i = 0; i < 32; ++i) {
-                const float fi = __shfl_sync(~0u, f, i);
-                if (s0 + i >= splits) break;
-                if (!live) continue;
-                const float2 x = *reinterpret_cast<const float2*>(rec + (size_t) (s0 + i) * ld + d);
-                v.x = fmaf(x.x, fi, v.x); v.y = fmaf(x.y, fi, v.y);
-            }
-        }
-        bf16* out = (bf16*) a.out + (size_t) row * g.out_ld() + h * g.vdim;
-        if (d < g.vdim) out[d] = __float2bfloat16_rn(v.x / den);
-        if (d + 1 < g.vdim) out[d + 1] = __float2bfloat16_rn(v.y / den);
+    den *= exp2f(s2 - top);
+    for (int s = lane; s < splits; s += 32) {
+        const float e = exp2f(rec[(size_t) s * ld + vcld] - top);
+        if (warp == 0) f[s] = e;
+        den = fmaf(rec[(size_t) s * ld + vcld + 1], e, den);
     }
+    den = skd::warp_sum(den);
+    __syncthreads();
+    for (int d = 2 * lane; d < vcld; d += 64) {
+        float2 v = make_float2(0.0f, 0.0f);
+#pragma unroll 8
+        for (int s = warp; s < splits; s += 4) {
+            const float2 x = *reinterpret_cast<const float2*>(rec + (size_t) s * ld + d);
+            v.x = fmaf(x.x, f[s], v.x); v.y = fmaf(x.y, f[s], v.y);
+        }
+        sum[warp * vcld + d] = v.x; sum[warp * vcld + d + 1] = v.y;
+    }
+    __syncthreads();
+    for (int d = threadIdx.x; d < g.vdim; d += 128)
+        ((bf16*) a.out)[(size_t) row * g.out_ld() + h * g.vdim + d] = __float2bfloat16_rn((sum[d] + sum[vcld + d] + sum[2 * vcld + d] + sum[3 * vcld + d]) / den);
 }
 
 // Pairs of a step's row reach no further than one row, so a decode step has a CTA row per sequence; prompts tile the pairs.
@@ -375,11 +375,11 @@ int32_t run_tile(const KvAttnArgs& a, cudaStream_t s) {
     const int seen = a.chunk > 0 ? std::min(a.kv_bound, a.chunk + (DECODE ? 0 : a.rows)) : a.kv_bound;
     const int64_t room = (int64_t) KV_PART_RECORDS / ((int64_t) a.rows * g.heads);
     const int want = (2 * sm_count() + mx * g.kv_heads - 1) / (mx * g.kv_heads);
-    int splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) want, (int64_t) (seen + TK - 1) / TK, room, 65535}));
+    int splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) want, (int64_t) (seen + TK - 1) / TK, room, 1024}));
     if (!DECODE && mx * g.kv_heads * 2 > sm_count()) splits = 1;
     SK_TRY(ensure_dynamic_smem((const void*) kv_attn_tile_kernel<KS, VN, DECODE>, bytes));
     SK_CUDA(launch_pdl(kv_attn_tile_kernel<KS, VN, DECODE>, dim3(mx, g.kv_heads, splits), dim3(S::WARPS * 32), bytes, s, a, splits));
-    if (splits > 1) SK_CUDA(launch_pdl(kv_merge_kernel, dim3(a.rows, (g.heads + 3) / 4), dim3(128), 0, s, a, splits));
+    if (splits > 1) SK_CUDA(launch_pdl(kv_merge_kernel, dim3(a.rows, g.heads), dim3(128), (splits + 4 * g.vcld()) * sizeof(float), s, a, splits));
     return SKAINET_CUDA_OK;
 }
 template <bool DECODE>

@@ -292,7 +292,7 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
     const int pos0 = a.map.pos[a.map.seq];
     const float skip = DELTA ? 0.0f : a.d[h];
     const bool holder = warp < 4;                                   // warps 0-3 hold the state, 4-7 the outputs
-    const int mt = warp & 3;                                        // the warp's 16 tokens
+    const int mt = holder ? warp : 7 - warp;                        // the warp's 16 tokens; later tokens sum over more, so the two kinds run opposite ways
 
     // state rows 16 (mt + 4 i) + gr (+ 8), columns 8 n + 2 tq (+ 1); left by an earlier pass
     float S[KT][NT][4];
@@ -392,14 +392,17 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
                 uint32_t f[4];
                 skd::ldsm4(f, a_at + ks * 32);
 #pragma unroll
-                for (int n = 0; n < NT; n += 2)
+                for (int n = 0; n < NT; n += 4) {                   // four sums in flight
+                    uint32_t bb[3][2][4];
 #pragma unroll
-                    for (int term = 2; term >= 0; --term) {
-                        uint32_t bb[4];
-                        skd::ldsm4_t(bb, s_at + term * s_term + bt_off + (ks * 16 * LV + n * 8) * 2);
-                        skd::mma_bf16(acc[n], f[0], f[1], f[2], f[3], bb[0], bb[1]);
-                        skd::mma_bf16(acc[n + 1], f[0], f[1], f[2], f[3], bb[2], bb[3]);
-                    }
+                    for (int j = 0; j < 3; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) skd::ldsm4_t(bb[j][e], s_at + j * s_term + bt_off + (ks * 16 * LV + (n + 2 * e) * 8) * 2);
+#pragma unroll
+                    for (int j = 2; j >= 0; --j)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) skd::mma_bf16(acc[n + e], f[0], f[1], f[2], f[3], bb[j][e >> 1][2 * (e & 1)], bb[j][e >> 1][2 * (e & 1) + 1]);
+                }
             }
         }
         float p[8][4];
@@ -428,16 +431,16 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
 #pragma unroll
                     for (int i = 0; i < 3; ++i) skd::ldsm4(f[i], t_at + ((i * CH + mt * 16 + lr + l8 * 8) * Z::LT + ks * 16 + l16 * 8) * 2);
 #pragma unroll
-                    for (int n = 0; n < NT; n += 2)
+                    for (int n = 0; n < NT; n += 4)
 #pragma unroll
                         for (int j = 2; j >= 0; --j) {
-                            uint32_t bb[4];
-                            skd::ldsm4_t(bb, w_at + j * Z::V_TERM + bt_off + (ks * 16 * LV + n * 8) * 2);
+                            uint32_t bb[2][4];
 #pragma unroll
-                            for (int i = 2 - j; i >= 0; --i) {
-                                skd::mma_bf16(acc[n], f[i][0], f[i][1], f[i][2], f[i][3], bb[0], bb[1]);
-                                skd::mma_bf16(acc[n + 1], f[i][0], f[i][1], f[i][2], f[i][3], bb[2], bb[3]);
-                            }
+                            for (int e = 0; e < 2; ++e) skd::ldsm4_t(bb[e], w_at + j * Z::V_TERM + bt_off + (ks * 16 * LV + (n + 2 * e) * 8) * 2);
+#pragma unroll
+                            for (int i = 2 - j; i >= 0; --i)
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) skd::mma_bf16(acc[n + e], f[i][0], f[i][1], f[i][2], f[i][3], bb[e >> 1][2 * (e & 1)], bb[e >> 1][2 * (e & 1) + 1]);
                         }
                 }
 #pragma unroll
@@ -494,23 +497,25 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
             }
 #pragma unroll
             for (int ks = 0; ks < CH / 16; ++ks)
+{
+                uint32_t f[KT][4];                                  // k transposed: rows are key coordinates
+#pragma unroll
+                for (int i = 0; i < KT; ++i) if (mt + 4 * i < ksn) skd::ldsm4_t(f[i], k + ((ks * 16 + lr + l16 * 8) * lk + 16 * (mt + 4 * i) + l8 * 8) * 2);
 #pragma unroll
                 for (int n = 0; n < NT; n += 2) {
                     uint32_t bb[3][4];
 #pragma unroll
                     for (int j = 0; j < 3; ++j) skd::ldsm4_t(bb[j], up_at + j * Z::V_TERM + bt_off + (ks * 16 * LV + n * 8) * 2);
 #pragma unroll
-                    for (int i = 0; i < KT; ++i) {
-                        if (mt + 4 * i >= ksn) break;
-                        uint32_t f[4];                              // k transposed: rows are key coordinates
-                        skd::ldsm4_t(f, k + ((ks * 16 + lr + l16 * 8) * lk + 16 * (mt + 4 * i) + l8 * 8) * 2);
+                    for (int j = 2; j >= 0; --j)
 #pragma unroll
-                        for (int j = 2; j >= 0; --j) {
-                            skd::mma_bf16(S[i][n], f[0], f[1], f[2], f[3], bb[j][0], bb[j][1]);
-                            skd::mma_bf16(S[i][n + 1], f[0], f[1], f[2], f[3], bb[j][2], bb[j][3]);
+                        for (int i = 0; i < KT; ++i) {
+                            if (mt + 4 * i >= ksn) break;
+                            skd::mma_bf16(S[i][n], f[i][0], f[i][1], f[i][2], f[i][3], bb[j][0], bb[j][1]);
+                            skd::mma_bf16(S[i][n + 1], f[i][0], f[i][1], f[i][2], f[i][3], bb[j][2], bb[j][3]);
                         }
-                    }
                 }
+            }
             put_state();
         } else {
 #pragma unroll
@@ -520,16 +525,16 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
                 skd::split3(p[2 * ks][0], p[2 * ks][1], f[0]); skd::split3(p[2 * ks][2], p[2 * ks][3], f[1]);
                 skd::split3(p[2 * ks + 1][0], p[2 * ks + 1][1], f[2]); skd::split3(p[2 * ks + 1][2], p[2 * ks + 1][3], f[3]);
 #pragma unroll
-                for (int n = 0; n < NT; n += 2)
+                for (int n = 0; n < NT; n += 4)
 #pragma unroll
                     for (int j = DELTA ? 2 : 0; j >= 0; --j) {
-                        uint32_t bb[4];
-                        skd::ldsm4_t(bb, (DELTA ? u_at + j * Z::V_TERM : v) + bt_off + (ks * 16 * LV + n * 8) * 2);
+                        uint32_t bb[2][4];
 #pragma unroll
-                        for (int i = 2 - j; i >= 0; --i) {
-                            skd::mma_bf16(acc[n], f[0][i], f[1][i], f[2][i], f[3][i], bb[0], bb[1]);
-                            skd::mma_bf16(acc[n + 1], f[0][i], f[1][i], f[2][i], f[3][i], bb[2], bb[3]);
-                        }
+                        for (int e = 0; e < 2; ++e) skd::ldsm4_t(bb[e], (DELTA ? u_at + j * Z::V_TERM : v) + bt_off + (ks * 16 * LV + (n + 2 * e) * 8) * 2);
+#pragma unroll
+                        for (int i = 2 - j; i >= 0; --i)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) skd::mma_bf16(acc[n + e], f[0][i], f[1][i], f[2][i], f[3][i], bb[e >> 1][2 * (e & 1)], bb[e >> 1][2 * (e & 1) + 1]);
                     }
             }
 #pragma unroll
