@@ -15,12 +15,13 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volati
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// x = sum of three bf16 terms, exact to fp32's 24 bits (while the last term does not underflow); two values per word.
+// x = sum of three bf16 terms of 8 bits each, exactly (while the last term does not underflow); two values per word.
 __device__ __forceinline__ void split3(float a, float b, uint32_t (&t)[3]) {
 #pragma unroll
     for (int i = 0; i < 3; ++i) {
-        t[i] = pack_bf16(a, b);
-        a -= bf16_lo(t[i]); b -= bf16_hi(t[i]);
+        const uint32_t x = __float_as_uint(a), y = __float_as_uint(b);
+        t[i] = __byte_perm(x, y, 0x7632);
+        a -= __uint_as_float(x & 0xffff0000u); b -= __uint_as_float(y & 0xffff0000u);
     }
 }
 

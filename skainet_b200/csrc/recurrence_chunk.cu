@@ -28,7 +28,7 @@ namespace {
 constexpr int CH = 64;                       // tokens of a chunk
 constexpr int CONV_ROWS = 16;
 
-int state_cols(const RecurGeom& g) { return !g.delta && g.vdim > 32 ? 64 : 32; }
+int state_cols(const RecurGeom& g) { return !g.delta && g.vdim > 32 && g.kdim <= 128 ? 64 : 32; }
 
 // Work buffers, all padded to whole chunks with zeros.
 struct Work {
@@ -191,6 +191,8 @@ __device__ __forceinline__ void decay_sums(float a, float b, int lane, double (&
     g[1] = s;
 }
 
+constexpr double MILD_DECAY = 50.0;          // a chunk's log decay up to which e^50 and e^-50 may be applied apart
+
 constexpr int INV_LD = CH + 4;
 // grid: (chunk, head); 128 threads
 __global__ void __launch_bounds__(128) recur_inverse_kernel(const RecurArgs a, const Work w) {
@@ -282,7 +284,7 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
     const RecurGeom& g = a.g;
     extern __shared__ __align__(16) uint8_t raw[];
     __shared__ double sG[2][CH];
-    __shared__ float s_step[2][CH], s_rq[2][CH], s_rk[2][CH], s_e[2][CH], s_f[2][CH];      // e^G, e^(G_end - G)
+    __shared__ float s_step[2][CH], s_rq[2][CH], s_rk[2][CH], s_e[2][CH], s_f[2][CH], s_col[2][CH];      // e^G, e^(G_end - G), the latter with |k|^-1 (and the step)
     const int kp = w.kp, lk = kp + 8, ksn = kp / 16, tiles = w.vp / VT, h = blockIdx.x / tiles, c0 = (blockIdx.x % tiles) * VT, grp = h / (g.heads / g.groups);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, tq = lane & 3, n_chunks = w.rows / CH;
     const uint32_t base = skd::smem_u32(raw), s_at = base + Z::STAGES * Z::stage(kp), up_at = s_at + 3 * kp * LV * 2, w_at = up_at + 3 * Z::V_TERM, u_at = w_at + 3 * Z::V_TERM;
@@ -345,6 +347,7 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
             const int t = 2 * lane + i;
             sG[b][t] = d[i]; s_step[b][t] = st[i]; s_rq[b][t] = rq[i]; s_rk[b][t] = rk[i];
             s_e[b][t] = expf((float) d[i]); s_f[b][t] = expf((float) (end - d[i]));
+            s_col[b][t] = s_f[b][t] * rk[i] * (DELTA ? 1.0f : st[i]);
         }
     };
     // three bf16 terms of a value pair into the terms' tiles
@@ -405,7 +408,7 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
                 }
             }
         }
-        float p[8][4];
+        float p[8][4], row0 = 0.0f, row1 = 0.0f;
         if (holder) {
             const float e0 = DELTA ? s_e[b][t0] * s_rk[b][t0] : 0.0f, e1 = DELTA ? s_e[b][t1] * s_rk[b][t1] : 0.0f, b0 = s_step[b][t0], b1 = s_step[b][t1];
             const float f0 = s_f[b][t0] * s_rk[b][t0], f1 = s_f[b][t1] * s_rk[b][t1];
@@ -468,19 +471,36 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
                     skd::mma_bf16(p[n + 1], f[0], f[1], f[2], f[3], bb[2], bb[3]);
                 }
             }
-            const double G0 = sG[b][t0], G1 = sG[b][t1];
-            const float r0 = s_rq[b][t0], r1 = s_rq[b][t1];
+            const double G0 = sG[b][t0], G1 = sG[b][t1], end = sG[b][CH - 1];
+            float e0, e1;                                           // factors of S^T q now, and of the outputs at the end
+            row0 = s_rq[b][t0]; row1 = s_rq[b][t1];
+            if (end > -MILD_DECAY) {
+                // e^(G_t - G_s) = e^(G_t - G_end) e^(G_end - G_s): a factor per column here and one per row at the end, both in range
 #pragma unroll
-            for (int n = 0; n < 8; ++n) {
-                if (n > 2 * mt + 1) break;
+                for (int n = 0; n < 8; ++n) {
+                    if (n > 2 * mt + 1) break;
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int s = n * 8 + tq * 2 + (i & 1), t = i < 2 ? t0 : t1;
-                    const float f = s <= t ? expf((float) ((i < 2 ? G0 : G1) - sG[b][s])) * (i < 2 ? r0 : r1) * s_rk[b][s] * (DELTA ? 1.0f : s_step[b][s]) : 0.0f;
-                    p[n][i] *= f;
+                    for (int i = 0; i < 2; ++i) {
+                        const int s = n * 8 + tq * 2 + i;
+                        const float f = s_col[b][s];
+                        p[n][i] *= s <= t0 ? f : 0.0f;
+                        p[n][i + 2] *= s <= t1 ? f : 0.0f;
+                    }
                 }
+                e0 = e1 = s_e[b][CH - 1];
+                row0 *= expf((float) (G0 - end)); row1 *= expf((float) (G1 - end));
+            } else {
+#pragma unroll
+                for (int n = 0; n < 8; ++n) {
+                    if (n > 2 * mt + 1) break;
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int s = n * 8 + tq * 2 + (i & 1), t = i < 2 ? t0 : t1;
+                        p[n][i] *= s <= t ? expf((float) ((i < 2 ? G0 : G1) - sG[b][s])) * s_rk[b][s] * (DELTA ? 1.0f : s_step[b][s]) : 0.0f;
+                    }
+                }
+                e0 = s_e[b][t0]; e1 = s_e[b][t1];
             }
-            const float e0 = s_e[b][t0] * r0, e1 = s_e[b][t1] * r1;
 #pragma unroll
             for (int n = 0; n < NT; ++n) { acc[n][0] *= e0; acc[n][1] *= e0; acc[n][2] *= e1; acc[n][3] *= e1; }
         }
@@ -547,8 +567,9 @@ __global__ void __launch_bounds__(256, 1) recur_scan_kernel(const RecurArgs a, c
                     uint32_t x = 0;
                     if (!DELTA) asm volatile("ld.shared.u32 %0, [%1];" : "=r"(x) : "r"(v + (t * LV + n * 8 + tq * 2) * 2));
                     const int col = c0 + n * 8 + tq * 2;
-                    if (col < g.vdim) out[col] = acc[n][2 * e] + skip * skd::bf16_lo(x);
-                    if (col + 1 < g.vdim) out[col + 1] = acc[n][2 * e + 1] + skip * skd::bf16_hi(x);
+                    const float f = e ? row1 : row0;
+                    if (col < g.vdim) out[col] = fmaf(acc[n][2 * e], f, skip * skd::bf16_lo(x));
+                    if (col + 1 < g.vdim) out[col + 1] = fmaf(acc[n][2 * e + 1], f, skip * skd::bf16_hi(x));
                 }
             }
             if (warp == 7 && c + 1 < n_chunks) store_scal(next, b ^ 1);
@@ -601,7 +622,7 @@ int32_t launch_recur_chunks(const RecurArgs& a, cudaStream_t s) {
         SK_CUDA(launch_pdl(recur_conv_kernel, dim3(w.rows / CONV_ROWS, 2 * g.groups + g.heads), dim3(256), conv_bytes, s, a, w));
     }
     if (!g.delta) {
-        if (state_cols(g) == 64) return w.kp <= 128 ? run_scan<false, 64, 2>(a, w, s) : run_scan<false, 64, 4>(a, w, s);
+        if (state_cols(g) == 64) return run_scan<false, 64, 2>(a, w, s);
         return w.kp <= 128 ? run_scan<false, 32, 2>(a, w, s) : run_scan<false, 32, 4>(a, w, s);
     }
     const int inv_bytes = CH * (w.kp + 8) * 2 + CH * INV_LD * 4;
