@@ -1,6 +1,6 @@
 // Ring attention with a chunk mask and a sink (contract: kv_attn.cuh).
 //
-//   kv_prep_kernel       biases, unit-rms queries and keys, ring append.
+//   kv_prep_kernel       biases, unit-rms queries and keys, ring append (prompts; in a decode step the tile kernel does it).
 //   kv_attn_tile_kernel  bf16: the MMA rows are (activation row, head) pairs that share a key/value head, so a staged key or value
 //                        row serves the whole group. In prompts each of four warps owns 16 pairs and all read the same tile of 64
 //                        keys; in a decode step four warps own the same 16 pairs and a quarter of the tile's keys each. Keys may
@@ -22,11 +22,11 @@ constexpr float NEG_BIG = -1e30f;            // maximum over no key: finite, so 
 // First position that position i sees.
 __device__ __forceinline__ int first_key(const KvAttnArgs& a, int i) { return a.chunk > 0 ? i / a.chunk * a.chunk : 0; }
 
-// One warp prepares one vector of a row: u < heads a query, u < heads + kv_heads a key, else a value.
-template <typename T>
-__device__ void prep_vector(const KvAttnArgs& a, int row, int u, int lane) {
+// One warp prepares one vector of a row: u < heads a query, u < heads + kv_heads a key, else a value; put(i, x) stores coordinate i.
+template <typename F>
+__device__ __forceinline__ void prep_vector(const KvAttnArgs& a, int row, int u, int lane, F&& put) {
     const KvGeom& g = a.g;
-    const bool is_q = u < g.heads, is_v = u >= g.heads + g.kv_heads;
+    const bool is_v = u >= g.heads + g.kv_heads;
     const int n = is_v ? g.vdim : g.dim, off = is_v ? (g.heads + g.kv_heads) * g.dim + (u - g.heads - g.kv_heads) * g.vdim : u * g.dim;
     const float *p = a.proj + (size_t) row * a.proj_ld + off, *b = a.bias ? a.bias + off : nullptr;
     float r = 1.0f;
@@ -35,14 +35,16 @@ __device__ void prep_vector(const KvAttnArgs& a, int row, int u, int lane) {
         for (int i = lane; i < n; i += 32) { const float v = p[i] + (b ? b[i] : 0.0f); ss = fmaf(v, v, ss); }
         r = 1.0f / sqrtf(skd::warp_sum(ss) / (float) n + a.eps);
     }
-    T* dst;
-    if (is_q) dst = (T*) a.q + ((size_t) row * g.heads + u) * g.kld();
-    else {
-        const int slot = a.map.pos_of(row) % a.cache.cap, kh = u - g.heads - (is_v ? g.kv_heads : 0);
-        const size_t at = ((size_t) a.map.seq_of(row) * g.kv_heads + kh) * a.cache.cap + slot;
-        dst = is_v ? (T*) a.cache.v + at * g.vcld() : (T*) a.cache.k + at * g.kld();
-    }
-    for (int i = lane; i < n; i += 32) skd::store_act(dst + i, (p[i] + (b ? b[i] : 0.0f)) * r);
+    for (int i = lane; i < n; i += 32) put(i, (p[i] + (b ? b[i] : 0.0f)) * r);
+}
+// Row of unit u >= heads in the ring.
+template <typename T>
+__device__ __forceinline__ T* cache_row(const KvAttnArgs& a, int row, int u) {
+    const KvGeom& g = a.g;
+    const bool is_v = u >= g.heads + g.kv_heads;
+    const int slot = a.map.pos_of(row) % a.cache.cap, kh = u - g.heads - (is_v ? g.kv_heads : 0);
+    const size_t at = ((size_t) a.map.seq_of(row) * g.kv_heads + kh) * a.cache.cap + slot;
+    return is_v ? (T*) a.cache.v + at * g.vcld() : (T*) a.cache.k + at * g.kld();
 }
 
 template <typename T>
@@ -50,7 +52,9 @@ __global__ void __launch_bounds__(256) kv_prep_kernel(const KvAttnArgs a) {
     skd::pdl_launch_dependents();
     skd::pdl_wait();
     const int units = a.g.heads + 2 * a.g.kv_heads, u = blockIdx.y * 8 + (threadIdx.x >> 5);
-    if (u < units) prep_vector<T>(a, blockIdx.x, u, threadIdx.x & 31);
+    if (u >= units) return;
+    T* dst = u < a.g.heads ? (T*) a.q + ((size_t) blockIdx.x * a.g.heads + u) * a.g.kld() : cache_row<T>(a, blockIdx.x, u);
+    prep_vector(a, blockIdx.x, u, threadIdx.x & 31, [&](int i, float x) { skd::store_act(dst + i, x); });
 }
 
 constexpr int RK = 128;                      // keys of a tile = threads of a CTA
@@ -137,7 +141,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     const int row_base = DECODE ? (int) blockIdx.x / tiles_m : 0, p0 = m_tile * S::ROWS, pairs = DECODE ? group : a.rows * group;
     const uint32_t sk = skd::smem_u32(raw), sv = sk + S::STAGES * TK * klds * 2, sq = S::Q_REGS ? sk + (S::STAGES - 1) * TK * klds * 2 : sv + S::STAGES * TK * vlds * 2;
     skd::pdl_launch_dependents();
-    skd::pdl_wait();
+    if (!DECODE) skd::pdl_wait();                                 // positions and the ring's older rows were left by earlier steps
     const int seq = a.map.seq_of(row_base);
     const bf16* kc = (const bf16*) a.cache.k + ((size_t) seq * g.kv_heads + kh) * a.cache.cap * kld;
     const bf16* vc = (const bf16*) a.cache.v + ((size_t) seq * g.kv_heads + kh) * a.cache.cap * vcld;
@@ -147,12 +151,13 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     int t0 = 0, t1 = (pos_last - lo) / TK + 1;
     if (splits > 1) { const int per = (t1 + splits - 1) / splits; t0 = min(t1, split * per); t1 = min(t1, t0 + per); }
 
-    auto load_tile = [&](int t, int stage) {
-        const int kch = kld / 8, both = kch + vcld / 8;
-        int slot = (lo + t * TK + warp) % a.cache.cap;              // a warp copies a key and its value
+    auto load_tile = [&](int t, int stage, int skip) {              // `skip`: a position that is not in the ring yet
+        const int kch = kld / 8, both = kch + vcld / 8, j0 = lo + t * TK;
+        int slot = (j0 + warp) % a.cache.cap;                       // a warp copies a key and its value
 #pragma unroll 4
         for (int r = warp; r < TK; r += S::WARPS) {
             for (int c = lane; c < both; c += 32) {
+                if (DECODE && j0 + r == skip) continue;
                 if (c < kch) skd::cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
                 else skd::cp16(sv + ((stage * TK + r) * vlds + (c - kch) * 8) * 2, vc + (size_t) slot * vcld + (c - kch) * 8);
             }
@@ -160,14 +165,36 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
             if (slot >= a.cache.cap) slot %= a.cache.cap;
         }
     };
-    // queries; rows past the last pair repeat it and are not stored
-    for (int i = threadIdx.x; i < S::ROWS * (kld / 8); i += S::WARPS * 32) {
-        const int r = i / (kld / 8), c = i % (kld / 8), p = min(p0 + r, pairs - 1);
-        skd::cp16(sq + (r * klds + c * 8) * 2, (const bf16*) a.q + ((size_t) (row_base + p / group) * g.heads + kh * group + p % group) * kld + c * 8);
-    }
+    // queries; rows past the last pair repeat it (prompts) or are zero, and are not stored
+    if (!DECODE)
+        for (int i = threadIdx.x; i < S::ROWS * (kld / 8); i += S::WARPS * 32) {
+            const int r = i / (kld / 8), c = i % (kld / 8), p = min(p0 + r, pairs - 1);
+            skd::cp16(sq + (r * klds + c * 8) * 2, (const bf16*) a.q + ((size_t) (row_base + p / group) * g.heads + kh * group + p % group) * kld + c * 8);
+        }
     skd::cp_commit();
 #pragma unroll
-    for (int s = 0; s < S::STAGES - 1; ++s) { if (t0 + s < t1) load_tile(t0 + s, s); skd::cp_commit(); }
+    for (int s = 0; s < S::STAGES - 1; ++s) { if (t0 + s < t1) load_tile(t0 + s, s, pos_last); skd::cp_commit(); }
+    if (DECODE) {
+        // the step's own vectors: biases and norms here, the new key and value into the ring and into the tile they belong to
+        skd::pdl_wait();
+        bf16* smem = (bf16*) raw;
+        const int new_tile = (pos_last - lo) / TK, new_row = (pos_last - lo) % TK;
+        const bool mine = new_tile >= t0 && new_tile < t1, staged = mine && new_tile < t0 + S::STAGES - 1;
+        for (int u = warp; u < S::ROWS + 2; u += S::WARPS) {
+            const int n = u == S::ROWS + 1 ? g.vdim : g.dim, np = u == S::ROWS + 1 ? vcld : kld;
+            if (u < S::ROWS) {
+                bf16* dst = smem + (sq - sk) / 2 + u * klds;
+                for (int i = lane; i < np; i += 32) if (p0 + u >= pairs || i >= n) dst[i] = __float2bfloat16_rn(0.0f);
+                if (p0 + u < pairs) prep_vector(a, row_base, kh * group + p0 + u, lane, [&](int i, float x) { dst[i] = __float2bfloat16_rn(x); });
+            } else if (mine) {
+                const int unit = g.heads + kh + (u == S::ROWS + 1 ? g.kv_heads : 0);
+                bf16 *ring = cache_row<bf16>(a, row_base, unit), *dst = nullptr;
+                if (staged) dst = u == S::ROWS ? smem + ((new_tile - t0) * TK + new_row) * klds : smem + (sv - sk) / 2 + ((new_tile - t0) * TK + new_row) * vlds;
+                prep_vector(a, row_base, unit, lane, [&](int i, float x) { ring[i] = __float2bfloat16_rn(x); if (dst) dst[i] = __float2bfloat16_rn(x); });
+                if (dst) for (int i = n + lane; i < np; i += 32) dst[i] = __float2bfloat16_rn(0.0f);
+            }
+        }
+    }
 
     const int wr = DECODE ? 0 : warp * 16;                        // the warp's first pair
     int pos_r[2], lo_r[2];
@@ -189,7 +216,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     const uint32_t v_at = sv + ((k0w + (lane & 7) + ((lane >> 3) & 1) * 8) * vlds + (lane >> 4) * 8) * 2;
     const float sc2 = a.scale * LOG2E;
     if (S::Q_REGS) {
-        skd::cp_wait<S::STAGES - 1>();
+        if (!DECODE) skd::cp_wait<S::STAGES - 1>();
         __syncthreads();
 #pragma unroll
         for (int k = 0; k < KS; ++k) if (k < ks_n) skd::ldsm4(qf[S::Q_REGS ? k : 0], q_at + k * 32);
@@ -200,7 +227,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
         const int stage = (t - t0) % S::STAGES;
         skd::cp_wait<S::STAGES - 2>();
         __syncthreads();
-        if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES);
+        if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES, -1);
         skd::cp_commit();
         float c[NK][4];
 #pragma unroll
@@ -408,9 +435,10 @@ int32_t run_prep(const KvAttnArgs& a, cudaStream_t s) {
 int32_t launch_kv_attention(const KvAttnArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return SKAINET_CUDA_OK;
     if (a.f32_act) { SK_TRY(run_prep<float>(a, s)); return run_rows<float>(a, s); }
+    const bool tiles = a.g.kld() <= 256 && a.g.vcld() <= 256;
+    if (tiles && a.map.seq < 0) return run_tile_size<true>(a, s);
     SK_TRY(run_prep<bf16>(a, s));
-    if (a.g.kld() > 256 || a.g.vcld() > 256) return run_rows<bf16>(a, s);
-    return a.map.seq < 0 ? run_tile_size<true>(a, s) : run_tile_size<false>(a, s);
+    return tiles ? run_tile_size<false>(a, s) : run_rows<bf16>(a, s);
 }
 
 }  // namespace sk

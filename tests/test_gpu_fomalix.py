@@ -90,9 +90,9 @@ def portions(m, t, cut, seq=0):
 # ---- mechanisms alone -------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("mixer", [
-    D(), D(heads=4, kv_heads=4, dim=128, vdim=128), D(heads=2, kv_heads=1, dim=48, vdim=200, conv=3), D(heads=8, kv_heads=2, dim=16, vdim=16, conv=2), D(heads=1, kv_heads=1, dim=3, vdim=5, conv=1),
-    S(), S(heads=4, groups=4, state=128, vdim=64, norm_groups=1), S(heads=2, groups=1, state=200, vdim=17, conv=2, norm_groups=2), S(heads=8, groups=2, state=16, vdim=64, conv=4, norm_groups=8), S(heads=1, groups=1, state=1, vdim=3, conv=1, norm_groups=1),
-    A(), A(heads=8, kv_heads=1, dim=128, vdim=128, chunk=64, scale=0.1), A(heads=5, kv_heads=5, dim=40, vdim=24, chunk=100, scale=0.4), A(heads=12, kv_heads=4, dim=64, vdim=192, chunk=150, scale=0.2), A(heads=1, kv_heads=1, dim=1, vdim=1, chunk=1, scale=1.0),
+    D(), D(heads=4, kv_heads=4, dim=128, vdim=128), D(heads=2, kv_heads=1, dim=48, vdim=200, conv=3), D(heads=8, kv_heads=2, dim=16, vdim=16, conv=2), D(heads=1, kv_heads=1, dim=3, vdim=5, conv=1), D(heads=1, kv_heads=1, dim=16, vdim=520), D(heads=2, kv_heads=2, dim=256, vdim=96),
+    S(), S(heads=4, groups=4, state=128, vdim=64, conv=4, norm_groups=1), S(heads=10, groups=2, state=16, vdim=64, conv=4, norm_groups=1), S(heads=3, groups=1, state=40, vdim=343, norm_groups=1), S(heads=4, groups=1, state=240, vdim=64, norm_groups=4), S(heads=2, groups=1, state=200, vdim=17, conv=2, norm_groups=2), S(heads=8, groups=2, state=16, vdim=64, conv=4, norm_groups=8), S(heads=1, groups=1, state=1, vdim=3, conv=1, norm_groups=1),
+    A(), A(heads=8, kv_heads=1, dim=128, vdim=128, chunk=64, scale=0.1), A(heads=5, kv_heads=5, dim=40, vdim=24, chunk=100, scale=0.4), A(heads=12, kv_heads=4, dim=64, vdim=192, chunk=150, scale=0.2), A(heads=40, kv_heads=2, dim=24, vdim=40, chunk=1000, scale=0.4), A(heads=1, kv_heads=1, dim=1, vdim=1, chunk=1, scale=1.0),
 ], ids=lambda m: f"{m[0]}-{'-'.join(str(v) for v in m[1].values() if not isinstance(v, dict))}")
 def test_one_mixer_in_prompts_and_decoding(make, dtype, mixer):
     """One layer without a feed-forward: whole prompts, then portions on both sides of every tile size, then single tokens."""
