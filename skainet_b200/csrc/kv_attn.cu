@@ -401,9 +401,15 @@ int32_t run_tile(const KvAttnArgs& a, cudaStream_t s) {
     const int mx = DECODE ? a.rows * ((group + 15) / 16) : (a.rows * group + S::ROWS - 1) / S::ROWS;
     const int seen = a.chunk > 0 ? std::min(a.kv_bound, a.chunk + (DECODE ? 0 : a.rows)) : a.kv_bound;
     const int64_t room = (int64_t) KV_PART_RECORDS / ((int64_t) a.rows * g.heads);
-    const int want = (2 * sm_count() + mx * g.kv_heads - 1) / (mx * g.kv_heads);
-    int splits = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) want, (int64_t) (seen + TK - 1) / TK, room, 1024}));
-    if (!DECODE && mx * g.kv_heads * 2 > sm_count()) splits = 1;
+    const int tiles = (seen + TK - 1) / TK, base = mx * g.kv_heads, slots = sm_count() * std::max(1, std::min(3, 227 * 1024 / (bytes + 1024)));
+    const int most = (int) std::max<int64_t>(1, std::min<int64_t>({(int64_t) tiles, room, (int64_t) (!DECODE && base * 2 > sm_count() ? 1 : 1024)}));
+    // rounds of resident CTAs, each as long as its tiles and a fixed part of about three tiles; a merge costs about as much once
+    int splits = 1;
+    int64_t best = INT64_MAX;
+    for (int k = 1; k <= most; ++k) {
+        const int64_t cost = ((int64_t) base * k + slots - 1) / slots * ((tiles + k - 1) / k + 3) + (k > 1 ? 3 : 0);
+        if (cost < best) { best = cost; splits = k; }
+    }
     SK_TRY(ensure_dynamic_smem((const void*) kv_attn_tile_kernel<KS, VN, DECODE>, bytes));
     SK_CUDA(launch_pdl(kv_attn_tile_kernel<KS, VN, DECODE>, dim3(mx, g.kv_heads, splits), dim3(S::WARPS * 32), bytes, s, a, splits));
     if (splits > 1) SK_CUDA(launch_pdl(kv_merge_kernel, dim3(a.rows, g.heads), dim3(128), (splits + 4 * g.vcld()) * sizeof(float), s, a, splits));
