@@ -12,6 +12,7 @@
 #include "tma.cuh"
 
 #include <algorithm>
+#include <climits>
 
 namespace sk {
 
@@ -152,17 +153,25 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
     if (splits > 1) { const int per = (t1 + splits - 1) / splits; t0 = min(t1, split * per); t1 = min(t1, t0 + per); }
 
     auto load_tile = [&](int t, int stage, int skip) {              // `skip`: a position that is not in the ring yet
-        const int kch = kld / 8, both = kch + vcld / 8, j0 = lo + t * TK;
-        int slot = (j0 + warp) % a.cache.cap;                       // a warp copies a key and its value
-#pragma unroll 4
-        for (int r = warp; r < TK; r += S::WARPS) {
-            for (int c = lane; c < both; c += 32) {
-                if (DECODE && j0 + r == skip) continue;
-                if (c < kch) skd::cp16(sk + ((stage * TK + r) * klds + c * 8) * 2, kc + (size_t) slot * kld + c * 8);
-                else skd::cp16(sv + ((stage * TK + r) * vlds + (c - kch) * 8) * 2, vc + (size_t) slot * vcld + (c - kch) * 8);
+        // a warp copies a key and its value at a time, a lane the same 16 bytes of each
+        const int kch = kld / 8, both = kch + vcld / 8, j0 = lo + t * TK, slot0 = j0 % a.cache.cap, hole = skip - j0;
+        for (int c = lane; c < both; c += 32) {
+            const bool is_k = c < kch;
+            const int ld = is_k ? kld : vcld, at = (is_k ? c : c - kch) * 8;
+            const bf16* src = (is_k ? kc : vc) + at;
+            uint32_t dst = is_k ? sk + ((stage * TK + warp) * klds + at) * 2 : sv + ((stage * TK + warp) * vlds + at) * 2;
+            const uint32_t dst_step = S::WARPS * (is_k ? klds : vlds) * 2;
+            if (slot0 + TK <= a.cache.cap) {
+                src += (size_t) (slot0 + warp) * ld;
+                const size_t src_step = (size_t) S::WARPS * ld;
+#pragma unroll
+                for (int r = 0; r < TK / S::WARPS; ++r, src += src_step, dst += dst_step)
+                    if (!DECODE || warp + r * S::WARPS != hole) skd::cp16(dst, src);
+            } else {
+#pragma unroll 1
+                for (int r = 0; r < TK / S::WARPS; ++r, dst += dst_step)
+                    if (!DECODE || warp + r * S::WARPS != hole) skd::cp16(dst, src + (size_t) ((slot0 + warp + r * S::WARPS) % a.cache.cap) * ld);
             }
-            slot += S::WARPS;
-            if (slot >= a.cache.cap) slot %= a.cache.cap;
         }
     };
     // queries; rows past the last pair repeat it (prompts) or are zero, and are not stored
@@ -227,7 +236,7 @@ kv_attn_tile_kernel(const KvAttnArgs a, int splits) {
         const int stage = (t - t0) % S::STAGES;
         skd::cp_wait<S::STAGES - 2>();
         __syncthreads();
-        if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES, -1);
+        if (t + S::STAGES - 1 < t1) load_tile(t + S::STAGES - 1, (t - t0 + S::STAGES - 1) % S::STAGES, INT_MIN / 2);
         skd::cp_commit();
         float c[NK][4];
 #pragma unroll
