@@ -33,7 +33,7 @@ typedef struct {
 typedef struct {
     int32_t n_layers, width, vocab;
     float eps, embed_scale;
-    int32_t loop_start, loop_stop, loop_times;   /* layers start .. stop - 1 run `times` times in a row, each pass with a cache of its own */
+    int32_t loop_start, loop_stop, loop_times;   /* the span [start, stop) of layers is gone through `times` times; 1: once, as the others */
     int32_t max_seq, max_batch;
     int32_t prefill_rows;     /* rows of one prompt pass; 0: the library's choice */
     int32_t act_f32;          /* 0: bf16 activations and cache, 32-bit accumulation and state; 1: everything in 32-bit */

@@ -6,7 +6,7 @@
 //   Mamba-2     z | x | B | C | dt                         ->  recurrence                   ->  gated norm ->  o
 //   x += norm1b(.), act = norm2(x)  ->  gate, up -> gelu * up -> down  ->  x += norm2b(.) [+ embedding output], act = next norm1(x)
 //
-// A layer of the looped span runs several times; every run has a cache or state of its own and shares the weights. The residual
+// The looped span is unrolled into layer runs: what a sequence holds belongs to a run, the weights to a layer. The residual
 // stream and all recurrent state are fp32; linears read a narrowed copy. Decode steps and prompt passes run the same body over
 // rows; only the row map and the kernels the row count selects differ.
 #include "decoder.cuh"

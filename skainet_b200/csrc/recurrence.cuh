@@ -33,7 +33,7 @@ struct RecurArgs {
     int proj_ld = 0, conv_off = 0;         // the convolution's channels are columns conv_off .. conv_off + conv_dim
     int q_off = 0, k_off = 0, v_off = 0;   // channels, counted from conv_off
     int dt_off = 0, beta_off = 0;          // columns of the decay's and of beta's pre-activations, one per head
-    const float *conv_w = nullptr, *conv_b = nullptr;     // [channel][taps], last column the current token's; [channel] or null
+    const float *conv_w = nullptr, *conv_b = nullptr;     // [channel][taps], oldest input first; [channel] or null
     const float *a_log = nullptr, *dt_bias = nullptr, *d = nullptr;
     float q_scale = 1.0f;
     float* state = nullptr;                // [sequence][head][kdim][vld]

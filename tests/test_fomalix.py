@@ -46,7 +46,7 @@ def test_the_delta_rule_replaces_what_a_key_held():
     v = np.array([[[3.0]], [[5.0]], [[7.0]]])
     one = np.ones((3, 1))
     o = F.delta_rule(k, k, v, one, one)
-    assert o[:, 0, 0].tolist() == [3.0, 5.0, 7.0]                       # the read-out sees the token's own write, which replaced 3
+    assert o[:, 0, 0].tolist() == [3.0, 5.0, 7.0]                       # a token reads what it just wrote; 7 took the place of 3
     o = F.delta_rule(k, k, v, 0.5 * one, 0.5 * one)
     np.testing.assert_allclose(o[:, 0, 0], [1.5, 2.5, 0.375 + 0.5 * (7 - 0.375)])
 
